@@ -35,6 +35,7 @@ extern "C" {
 
 #define ARCB_ACT_F16 0  /* 16-bit activations held as IEEE half (default)     */
 #define ARCB_ACT_BF16 1 /* 16-bit activations held as bfloat16                */
+#define ARCB_ACT_F32 2  /* 32-bit everywhere, CUDA-core products (layered engines only) */
 
 #define ARCB_GEMM_AUTO 0 /* tcgen05 GEMM wherever the shape allows (K % 64 == 0)   */
 #define ARCB_GEMM_SIMT 1 /* CUDA-core GEMM everywhere (debug cross-check)      */
@@ -119,6 +120,83 @@ int arcb_engine_load_tensor(arcb_engine* eng, int32_t kind, int32_t layer, const
  * and ARCB_ACT_BF16 should be used instead.  No counterpart in the reference (which runs bf16). */
 int arcb_engine_saturation_count(arcb_engine* eng, int64_t* count, int32_t reset, void* stream);
 
+/* ---- layered engines: models described as a list of layers ------------- *
+ * A layered engine is the same handle as above with the network given as data: per layer a token
+ * mixer (softmax attention or a matrix-memory recurrence) and an optional feed-forward.  Sessions,
+ * prefill, decode, polling and sampling are the same entry points for both kinds of engine.  No
+ * counterpart in the reference, whose only network is TinyTransformer. */
+
+#define ARCB_MIXER_ATTENTION 0 /* causal softmax attention, H query heads on G key/value heads          */
+#define ARCB_MIXER_MLSTM 1     /* matrix memory with exponential input gate and stabiliser (mLSTM)      */
+
+#define ARCB_MLP_NONE 0
+#define ARCB_MLP_RELU2 1       /* W_down relu(W_up x)^2                                                 */
+
+#define ARCB_NORM_RMS 0
+#define ARCB_NORM_LAYER 1      /* centred, gain only                                                    */
+
+typedef struct arcb_layer_desc {
+  int32_t mixer;        /* ARCB_MIXER_*                                                                 */
+  int32_t heads;        /* query heads (attention) / memory heads (mLSTM)                               */
+  int32_t kv_heads;     /* attention: key/value heads, divides heads                                    */
+  int32_t dim, vdim;    /* per-head query/key and value size, 1..256                                    */
+  int32_t kv_from;      /* attention: layer whose cached keys and values are read, -1 = its own         */
+  int32_t qkv_bias;     /* projections of q, k and v have biases                                        */
+  int32_t qk_norm;      /* per-head RMS norm of queries and keys                                        */
+  int32_t sink;         /* softmax denominator also holds exp(sink[head])                               */
+  int32_t out_gate;     /* concatenated heads are multiplied by sigmoid(W_g x)                          */
+  float scale;          /* attention: factor of q.k                                                     */
+  float q_temp_coef;    /* query gain 1 + coef * ln(floor((p + 1) / every) + 1); every 0 = none         */
+  int32_t q_temp_every;
+  float gate_cap;       /* mLSTM: gates are cap * tanh(. / cap)                                         */
+  int32_t mlp;          /* ARCB_MLP_*                                                                   */
+  int32_t d_ff;
+} arcb_layer_desc;
+
+/* Norms sit AFTER the residual sum: x <- norm1(alpha x + mixer(x)), x <- norm2(alpha x + mlp(x)). */
+typedef struct arcb_model_desc {
+  int32_t width, vocab, n_layers;
+  int32_t norm;         /* ARCB_NORM_*, all norms of the residual stream                                */
+  int32_t act_format;   /* ARCB_ACT_*                                                                   */
+  int32_t gemm_path;    /* ARCB_GEMM_AUTO / ARCB_GEMM_SIMT                                              */
+  int32_t attn_path;    /* ARCB_ATTN_AUTO / ARCB_ATTN_STREAM (prefill through the streaming kernel)     */
+  int32_t mlstm_path;   /* ARCB_MLSTM_AUTO / ARCB_MLSTM_STEP                                            */
+  int32_t fused_proj;   /* 1: head norms, gates and cache writes inside the projection GEMM             */
+  float norm_eps, residual_alpha, logit_scale;
+} arcb_model_desc;
+#define ARCB_MLSTM_AUTO 0 /* chunkwise tensor-core prefill where the sizes allow                        */
+#define ARCB_MLSTM_STEP 1 /* token-by-token recurrence for prefill as well                              */
+
+/* Tensor kinds of a layered engine (arcb_engine_load_tensor, fp32 sources in [out, in] order). */
+enum arcb_lm_tensor_kind {
+  ARCB_L_EMBED = 0,   /* [vocab, width]                                  */
+  ARCB_L_FINAL_NORM,  /* [width]                                         */
+  ARCB_L_HEAD,        /* [vocab, width]                                  */
+  ARCB_L_NORM1,       /* [width] per layer, from here on                 */
+  ARCB_L_NORM2,
+  ARCB_L_Q,           /* [heads * dim, width]                            */
+  ARCB_L_Q_B,
+  ARCB_L_K,           /* [kv_heads * dim, width] (mLSTM: heads * dim)    */
+  ARCB_L_K_B,
+  ARCB_L_V,           /* [kv_heads * vdim, width] (mLSTM: heads * vdim)  */
+  ARCB_L_V_B,
+  ARCB_L_G,           /* [heads * vdim, width]                           */
+  ARCB_L_O,           /* [width, heads * vdim]                           */
+  ARCB_L_Q_NORM,      /* [dim]                                           */
+  ARCB_L_K_NORM,      /* [dim]                                           */
+  ARCB_L_SINK,        /* [heads]                                         */
+  ARCB_L_HEAD_NORM,   /* [heads * vdim]                                  */
+  ARCB_L_I,           /* [heads, width]                                  */
+  ARCB_L_I_B,
+  ARCB_L_F,
+  ARCB_L_F_B,
+  ARCB_L_UP,          /* [d_ff, width]                                   */
+  ARCB_L_DOWN,        /* [width, d_ff]                                   */
+  ARCB_L_COUNT
+};
+
+int arcb_engine_create_layered(const arcb_model_desc* model, const arcb_layer_desc* layers, arcb_engine** out);
+
 /* ---- session: one batch of sequences sharing a static KV cache --------- */
 
 /* StaticKVCache + GridStateUpdater + the per-call tensors of generate_output
@@ -164,6 +242,10 @@ typedef struct arcb_session_desc {
   int32_t top_k;
   uint64_t sample_seed;
   const int32_t* d_sample_stream; /* optional int32 [B] */
+  int32_t end_token;              /* layered engines: token that finishes a row, < 0 = none (the
+                                     grid model's END is fixed).  d_step_logits is then
+                                     [B][max_new][vocab], and the cache buffer holds per layer either
+                                     keys and values or the recurrent state of every sequence     */
 } arcb_session_desc;
 
 int64_t arcb_session_workspace_bytes(const arcb_engine* eng, int32_t n_seqs,
@@ -217,6 +299,19 @@ typedef struct arcb_prefill_args {
   const int32_t* d_grid_y;     /*           (src/inference.py:171-221)         */
   const int32_t* d_grid_in_output;
   float* d_first_logits;       /* optional [n_first][14]                       */
+  /* Layered engines: the rows of one sequence are consecutive and continue where its cache and state
+   * end (kv_slot = position, kv_count = position + 1; a segment at position 0 starts the sequence
+   * afresh).  d_pos_xyz, the K/V scratch fields and the grid fields are not read; d_prompt_len is the
+   * number of positions cached after the call; logits are [rows][vocab]. */
+  int32_t n_segs;
+  const int32_t* d_seg_row0;   /* [n_segs] first packed row                    */
+  const int32_t* d_seg_rows;   /* [n_segs]                                     */
+  const int32_t* d_seg_seq;    /* [n_segs] cache row                           */
+  const int32_t* d_seg_pos0;   /* [n_segs] position of the first row           */
+  int32_t n_logit_rows;        /* rows whose logits are wanted without arming the decode loop */
+  const int32_t* d_logit_row;  /* [n_logit_rows]                               */
+  float* d_logits;             /* [n_logit_rows][vocab]                        */
+  float* d_residuals;          /* optional [n_layers][n_tokens][width]: residual stream after every layer */
 } arcb_prefill_args;
 
 int arcb_prefill(arcb_session* s, const arcb_prefill_args* a, void* stream);
@@ -225,6 +320,20 @@ int arcb_prefill(arcb_session* s, const arcb_prefill_args* a, void* stream);
  * GridStateUpdater.update -> _decode_step -> argmax -> finished/END handling,
  * each iteration one replay of a CUDA graph captured on first use. */
 int arcb_decode(arcb_session* s, int32_t n_steps, void* stream);
+
+/* Layered engines: a sequence that has produced max_new tokens counts as finished and is held.
+ *
+ * arcb_session_feed names the sequences and tokens of the next arcb_decode step (teacher forcing a
+ * subset of the slots: all other sequences hold still, their cache and state untouched). */
+int arcb_session_feed(arcb_session* s, int32_t n, const int32_t* d_seqs, const int32_t* d_tokens, void* stream);
+
+/* Layered engines: device address of the last decode step's logits, fp32 rows of *pitch floats
+ * indexed by sequence; valid until the session's next call. */
+int arcb_session_step_logits(arcb_session* s, float** d_logits, int32_t* pitch);
+
+/* Layered engines: synchronises `stream` and copies one flag per sequence to the host: 1 = the sequence has
+ * emitted end_token or used up max_new (it is held then). */
+int arcb_session_finished(arcb_session* s, int32_t* h_finished, void* stream);
 
 /* Synchronises `stream`, then reports how many rows have emitted END and the
  * device error word (0 = none). Replaces `finished.all()` (src/inference.py:594). */

@@ -9,7 +9,7 @@ from pathlib import Path
 
 LIB_PATH = Path(__file__).resolve().parent / "libarcb200.so"
 
-ACT_F16, ACT_BF16 = 0, 1
+ACT_F16, ACT_BF16, ACT_F32 = 0, 1, 2
 GEMM_AUTO, GEMM_SIMT, GEMM_TC, GEMM_TC_1CTA, GEMM_TC_2CTA = 0, 1, 2, 3, 4
 ATTN_AUTO, ATTN_STREAM = 0, 1
 
@@ -22,10 +22,22 @@ TENSOR_KINDS = [
 ]
 KIND = {name: i for i, name in enumerate(TENSOR_KINDS)}
 
+# layered engines (enum arcb_lm_tensor_kind and the mixer / feed-forward / norm codes)
+LAYERED_KINDS = [
+    "EMBED", "FINAL_NORM", "HEAD", "NORM1", "NORM2", "Q", "Q_B", "K", "K_B", "V", "V_B", "G", "O",
+    "Q_NORM", "K_NORM", "SINK", "HEAD_NORM", "I", "I_B", "F", "F_B", "UP", "DOWN",
+]
+LAYERED_KIND = {name: i for i, name in enumerate(LAYERED_KINDS)}
+MIXERS = {"attention": 0, "mlstm": 1}
+MLPS = {None: 0, "relu2": 1}
+NORMS = {"rms": 0, "layer": 1}
+MLSTM_AUTO, MLSTM_STEP = 0, 1
+
 EXPORTS = [
     "arcb_last_error", "arcb_device_ok", "arcb_engine_create", "arcb_engine_destroy",
     "arcb_engine_load_tensor", "arcb_session_workspace_bytes", "arcb_kv_cache_bytes",
     "arcb_session_create", "arcb_session_destroy", "arcb_prefill", "arcb_decode",
+    "arcb_engine_create_layered", "arcb_session_feed", "arcb_session_step_logits", "arcb_session_finished",
     "arcb_session_poll", "arcb_engine_saturation_count", "arcb_session_attention_probe", "arcb_launch_count", "arcb_op_rmsnorm", "arcb_op_gemm",
     "arcb_op_gemm_residual", "arcb_gemm_splitk_scratch_bytes", "arcb_op_gemm_residual_splitk",
     "arcb_attn_scratch_bytes", "arcb_op_decode_attention", "arcb_op_decode_attention_static",
@@ -54,7 +66,7 @@ class SessionDesc(C.Structure):
         ("d_palette_mask", C.c_void_p), ("d_target_shape", C.c_void_p),
         ("palette_penalty", C.c_float), ("shape_penalty", C.c_float), ("disallow_token_mask", C.c_uint32),
         ("temperature", C.c_float), ("top_k", C.c_int32), ("sample_seed", C.c_uint64),
-        ("d_sample_stream", C.c_void_p),
+        ("d_sample_stream", C.c_void_p), ("end_token", C.c_int32),
     ]
 
 
@@ -70,6 +82,26 @@ class PrefillArgs(C.Structure):
         ("n_first", C.c_int32), ("d_first_row", C.c_void_p), ("d_first_seq", C.c_void_p),
         ("d_prompt_len", C.c_void_p), ("d_grid_x", C.c_void_p), ("d_grid_y", C.c_void_p),
         ("d_grid_in_output", C.c_void_p), ("d_first_logits", C.c_void_p),
+        ("n_segs", C.c_int32), ("d_seg_row0", C.c_void_p), ("d_seg_rows", C.c_void_p), ("d_seg_seq", C.c_void_p),
+        ("d_seg_pos0", C.c_void_p), ("n_logit_rows", C.c_int32), ("d_logit_row", C.c_void_p),
+        ("d_logits", C.c_void_p), ("d_residuals", C.c_void_p),
+    ]
+
+
+class LayerDesc(C.Structure):
+    _fields_ = [
+        ("mixer", C.c_int32), ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32),
+        ("kv_from", C.c_int32), ("qkv_bias", C.c_int32), ("qk_norm", C.c_int32), ("sink", C.c_int32),
+        ("out_gate", C.c_int32), ("scale", C.c_float), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_int32),
+        ("gate_cap", C.c_float), ("mlp", C.c_int32), ("d_ff", C.c_int32),
+    ]
+
+
+class ModelDesc(C.Structure):
+    _fields_ = [
+        ("width", C.c_int32), ("vocab", C.c_int32), ("n_layers", C.c_int32), ("norm", C.c_int32),
+        ("act_format", C.c_int32), ("gemm_path", C.c_int32), ("attn_path", C.c_int32), ("mlstm_path", C.c_int32),
+        ("fused_proj", C.c_int32), ("norm_eps", C.c_float), ("residual_alpha", C.c_float), ("logit_scale", C.c_float),
     ]
 
 
@@ -128,6 +160,10 @@ def load() -> C.CDLL:
     lib.arcb_kv_cache_bytes.argtypes = [vp, i32, i32]
     lib.arcb_session_create.argtypes = [vp, C.POINTER(SessionDesc), C.POINTER(vp)]
     lib.arcb_session_destroy.argtypes = [vp]
+    lib.arcb_engine_create_layered.argtypes = [C.POINTER(ModelDesc), C.POINTER(LayerDesc), C.POINTER(vp)]
+    lib.arcb_session_feed.argtypes = [vp, i32, vp, vp, vp]
+    lib.arcb_session_step_logits.argtypes = [vp, C.POINTER(vp), C.POINTER(i32)]
+    lib.arcb_session_finished.argtypes = [vp, vp, vp]
     lib.arcb_prefill.argtypes = [vp, C.POINTER(PrefillArgs), vp]
     lib.arcb_decode.argtypes = [vp, i32, vp]
     lib.arcb_session_poll.argtypes = [vp, C.POINTER(i32), C.POINTER(i32), vp]

@@ -81,6 +81,36 @@ __device__ __forceinline__ uint32_t pack2_bf16(float a, float b) {
   return *reinterpret_cast<uint32_t*>(&h);
 }
 
+// ---- activation elements in any of the three formats (0 = bfloat16, 1 = IEEE half, 2 = fp32) ----
+__host__ __device__ __forceinline__ int act_bytes(int fmt) { return fmt == 2 ? 4 : 2; }
+
+__device__ __forceinline__ float4 ld_act4(const void* base, size_t idx, int fmt) {
+  if (fmt == 2) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(base) + idx);
+  const uint2 r = *reinterpret_cast<const uint2*>(reinterpret_cast<const uint16_t*>(base) + idx);
+  const float2 a = unpack2_act(r.x, fmt), b = unpack2_act(r.y, fmt);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void st_act4(void* base, size_t idx, float4 v, int fmt) {
+  if (fmt == 2) {
+    *reinterpret_cast<float4*>(reinterpret_cast<float*>(base) + idx) = v;
+  } else {
+    uint2 r;
+    r.x = pack2_act(v.x, v.y, fmt);
+    r.y = pack2_act(v.z, v.w, fmt);
+    *reinterpret_cast<uint2*>(reinterpret_cast<uint16_t*>(base) + idx) = r;
+  }
+}
+__device__ __forceinline__ float ld_act(const void* base, size_t idx, int fmt) {
+  if (fmt == 2) return reinterpret_cast<const float*>(base)[idx];
+  if (fmt == 1) return __half2float(reinterpret_cast<const __half*>(base)[idx]);
+  return __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(base)[idx]);
+}
+__device__ __forceinline__ void st_act(void* base, size_t idx, float v, int fmt) {
+  if (fmt == 2) reinterpret_cast<float*>(base)[idx] = v;
+  else if (fmt == 1) reinterpret_cast<__half*>(base)[idx] = __float2half_rn(fminf(fmaxf(v, -65504.f), 65504.f));
+  else reinterpret_cast<__nv_bfloat16*>(base)[idx] = __float2bfloat16_rn(v);
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

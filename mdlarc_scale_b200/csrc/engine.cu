@@ -13,6 +13,7 @@
 #include "attn_stream.cuh"
 #include "gemm.cuh"
 #include "launch.cuh"
+#include "engine.cuh"
 #include "rowops.cuh"
 
 // ---------------------------------------------------------------------------
@@ -45,97 +46,13 @@ bool arcb_pdl_suppressed() { return g_pdl_suppress; }
 
 void arcb_set_last_error(const char* msg) { g_last_error = msg ? msg : ""; }
 
-static int fail(int code, const char* msg) {
+int arcb_fail(int code, const char* msg) {
   g_last_error = msg;
   return code;
 }
-static int fail_cuda(cudaError_t e, const char* where) {
+int arcb_fail_cuda(cudaError_t e, const char* where) {
   g_last_error = std::string(where) + ": " + cudaGetErrorString(e);
   return (int)e;
-}
-#define CK(call)                                         \
-  do {                                                   \
-    cudaError_t e__ = (call);                            \
-    if (e__ != cudaSuccess) return fail_cuda(e__, #call); \
-  } while (0)
-#define CKL(expr, what)                                            \
-  do {                                                             \
-    int r__ = (expr);                                              \
-    if (r__ != 0) {                                                \
-      if (r__ > 0 && r__ < 1000) return fail_cuda((cudaError_t)r__, what); \
-      return fail(r__ < 0 ? ARCB_E_ARG : r__, what);              \
-    }                                                              \
-  } while (0)
-
-// GEMM weights hold the bf16-rounded parameter values in the 16-bit container of the activations
-// (half or bfloat16), because the tensor-core MMA needs both operands in one format.
-struct LayerWeights {
-  float* ln1_w = nullptr;
-  uint16_t* w_qkv = nullptr;   // [3d][d]
-  uint16_t* w_out = nullptr;   // [d][d]
-  float* ln2_w = nullptr;
-  uint16_t* w_gu = nullptr;    // [2 dff][d], 64 gate rows then the matching 64 up rows, repeated
-  float* b_gu = nullptr;       // [2 dff] packed the same way
-  uint16_t* w_down = nullptr;  // [d][dff]
-  float* b_down = nullptr;          // [d]
-};
-
-struct arcb_engine {
-  arcb_config cfg;
-  int device = 0;
-  std::vector<LayerWeights> layers;
-  float* token_embed = nullptr;
-  float* example_embed = nullptr;
-  float* lnf_w = nullptr;
-  float* lm_head = nullptr;
-  float* rope = nullptr;  // cos_x | sin_x | cos_y | sin_y | cos_z | sin_z
-  int* d_err = nullptr;
-  std::vector<void*> allocs;
-  std::vector<char> loaded;  // [ARCB_T_COUNT * max(L,1)]
-  bool act_f16() const { return cfg.act_format == ARCB_ACT_F16; }
-};
-
-struct arcb_session {
-  arcb_engine* eng = nullptr;
-  arcb_session_desc desc;
-  int splits = 1;
-  // workspace carve-up
-  float* x = nullptr;
-  uint16_t* xn16 = nullptr;
-  uint16_t* q16 = nullptr;
-  uint16_t* attn16 = nullptr;
-  uint16_t* h16 = nullptr;
-  uint16_t* k16 = nullptr;  // K/V of one prefill call in the activation format
-  uint16_t* v16 = nullptr;
-  float* attn_scratch = nullptr;
-  float* gemm_scratch = nullptr;   // split-K partials of the decode step's residual GEMMs
-  int* example_ids = nullptr;
-  bool use_examples = false;
-  DecodeState st{};
-  cudaGraph_t graph = nullptr;
-  cudaGraphExec_t graph_exec = nullptr;
-  cudaStream_t capture_stream = nullptr;
-  long long graph_kernels = 0;
-  bool armed = false;
-  // event pair recorded (as graph nodes) around the layer-0 decode-attention launch of every replay
-  cudaEvent_t probe_begin = nullptr, probe_end = nullptr;
-  bool probe_recorded = false;
-  // the integer state block is cleared by the first arcb_prefill, on that call's stream
-  int* state_ints = nullptr;
-  size_t n_state_ints = 0;
-  bool state_cleared = false;
-};
-
-static size_t align_up(size_t v, size_t a) { return (v + a - 1) / a * a; }
-
-template <typename T>
-static int dev_alloc(arcb_engine* e, T** out, size_t count) {
-  void* p = nullptr;
-  cudaError_t r = cudaMalloc(&p, count * sizeof(T));
-  if (r != cudaSuccess) return (int)r;
-  e->allocs.push_back(p);
-  *out = reinterpret_cast<T*>(p);
-  return 0;
 }
 
 extern "C" const char* arcb_last_error(void) { return g_last_error.c_str(); }
@@ -156,15 +73,17 @@ extern "C" int64_t arcb_launch_count(int reset) {
 // engine
 // ---------------------------------------------------------------------------
 extern "C" int arcb_engine_create(const arcb_config* cfg, arcb_engine** out) {
-  if (!cfg || !out) return fail(ARCB_E_ARG, "null argument");
-  if (cfg->vocab_size != ARCB_VOCAB) return fail(ARCB_E_UNSUPPORTED, "vocab_size must be 14");
+  if (!cfg || !out) return arcb_fail(ARCB_E_ARG, "null argument");
+  if (cfg->act_format != ARCB_ACT_F16 && cfg->act_format != ARCB_ACT_BF16)
+    return arcb_fail(ARCB_E_UNSUPPORTED, "act_format must be half or bfloat16");
+  if (cfg->vocab_size != ARCB_VOCAB) return arcb_fail(ARCB_E_UNSUPPORTED, "vocab_size must be 14");
   if (cfg->n_heads <= 0 || cfg->d_model != cfg->n_heads * ARCB_HEAD_DIM)
-    return fail(ARCB_E_UNSUPPORTED, "head_dim must be 64");
+    return arcb_fail(ARCB_E_UNSUPPORTED, "head_dim must be 64");
   if (cfg->d_model % 128 || cfg->d_ff % 64 || cfg->n_layers <= 0 || cfg->d_ff <= 0)
-    return fail(ARCB_E_UNSUPPORTED, "d_model must be a multiple of 128 and d_ff of 64");
+    return arcb_fail(ARCB_E_UNSUPPORTED, "d_model must be a multiple of 128 and d_ff of 64");
   if (cfg->max_x <= 0 || cfg->max_y <= 0 || cfg->max_z <= 0 || cfg->num_examples <= 0)
-    return fail(ARCB_E_ARG, "bad table extents");
-  if (!arcb_device_ok()) return fail(ARCB_E_UNSUPPORTED, "current device is not compute capability 10.x");
+    return arcb_fail(ARCB_E_ARG, "bad table extents");
+  if (!arcb_device_ok()) return arcb_fail(ARCB_E_UNSUPPORTED, "current device is not compute capability 10.x");
   CKL(arcb_gemm_init(), "gemm init (shared-memory opt-in / cuTensorMapEncodeTiled lookup)");
   CKL(arcb_attn_prefill_init(), "prefill attention init (shared-memory opt-in)");
   arcb_engine* e = new arcb_engine();
@@ -194,7 +113,7 @@ extern "C" int arcb_engine_create(const arcb_config* cfg, arcb_engine** out) {
   r |= dev_alloc(e, &e->d_err, 64);
   if (r) {
     arcb_engine_destroy(e);
-    return fail(ARCB_E_STATE, "cudaMalloc of packed weights failed");
+    return arcb_fail(ARCB_E_STATE, "cudaMalloc of packed weights failed");
   }
   cudaMemset(e->d_err, 0, 64 * sizeof(int));
   *out = e;
@@ -203,6 +122,7 @@ extern "C" int arcb_engine_create(const arcb_config* cfg, arcb_engine** out) {
 
 extern "C" int arcb_engine_destroy(arcb_engine* e) {
   if (!e) return ARCB_OK;
+  if (e->lm) lm_destroy(e->lm);
   for (void* p : e->allocs) cudaFree(p);
   delete e;
   return ARCB_OK;
@@ -210,13 +130,14 @@ extern "C" int arcb_engine_destroy(arcb_engine* e) {
 
 extern "C" int arcb_engine_load_tensor(arcb_engine* e, int32_t kind, int32_t layer, const float* src,
                                        int64_t numel, void* stream_v) {
-  if (!e || !src) return fail(ARCB_E_ARG, "null argument");
-  if (kind < 0 || kind >= ARCB_T_COUNT) return fail(ARCB_E_ARG, "unknown tensor kind");
+  if (!e || !src) return arcb_fail(ARCB_E_ARG, "null argument");
+  if (e->lm) return lm_load_tensor(e, kind, layer, src, numel, (cudaStream_t)stream_v);
+  if (kind < 0 || kind >= ARCB_T_COUNT) return arcb_fail(ARCB_E_ARG, "unknown tensor kind");
   cudaStream_t stream = (cudaStream_t)stream_v;
   const arcb_config& c = e->cfg;
   const long long d = c.d_model, dff = c.d_ff;
   const bool per_layer = kind >= ARCB_T_LN1_W && kind <= ARCB_T_DOWN_B;
-  if (per_layer && (layer < 0 || layer >= c.n_layers)) return fail(ARCB_E_ARG, "layer out of range");
+  if (per_layer && (layer < 0 || layer >= c.n_layers)) return arcb_fail(ARCB_E_ARG, "layer out of range");
   LayerWeights* L = per_layer ? &e->layers[layer] : nullptr;
   long long rows = 0, cols = 0;
   void* dst = nullptr;
@@ -245,9 +166,9 @@ extern "C" int arcb_engine_load_tensor(arcb_engine* e, int32_t kind, int32_t lay
     case ARCB_T_ROPE_SIN_Y: rows = 1; cols = ny; dst = e->rope + 2 * nx + ny; break;
     case ARCB_T_ROPE_COS_Z: rows = 1; cols = nz; dst = e->rope + 2 * nx + 2 * ny; break;
     case ARCB_T_ROPE_SIN_Z: rows = 1; cols = nz; dst = e->rope + 2 * nx + 2 * ny + nz; break;
-    default: return fail(ARCB_E_ARG, "unknown tensor kind");
+    default: return arcb_fail(ARCB_E_ARG, "unknown tensor kind");
   }
-  if (numel != rows * cols) return fail(ARCB_E_ARG, "tensor has the wrong number of elements");
+  if (numel != rows * cols) return arcb_fail(ARCB_E_ARG, "tensor has the wrong number of elements");
   if (kind >= ARCB_T_ROPE_COS_X) {
     CK(cudaMemcpyAsync(dst, src, (size_t)numel * sizeof(float), cudaMemcpyDeviceToDevice, stream));
   } else {
@@ -260,6 +181,7 @@ extern "C" int arcb_engine_load_tensor(arcb_engine* e, int32_t kind, int32_t lay
 }
 
 static bool engine_complete(const arcb_engine* e) {
+  if (e->lm) return lm_complete(e);
   const int L = e->cfg.n_layers;
   for (int k = 0; k < ARCB_T_COUNT; ++k) {
     const bool per_layer = k >= ARCB_T_LN1_W && k <= ARCB_T_DOWN_B;
@@ -324,27 +246,44 @@ static WsLayout ws_layout(const arcb_engine* e, int B, int P, int splits) {
 extern "C" int64_t arcb_session_workspace_bytes(const arcb_engine* e, int32_t n_seqs,
                                                 int32_t max_prefill_tokens, int32_t attn_splits) {
   if (!e || n_seqs <= 0 || max_prefill_tokens < 0) return -1;
+  if (e->lm) return lm_workspace_bytes(e, n_seqs, max_prefill_tokens, attn_splits);
   return (int64_t)ws_layout(e, n_seqs, max_prefill_tokens, choose_splits(e, n_seqs, attn_splits)).total;
 }
 
 extern "C" int64_t arcb_kv_cache_bytes(const arcb_engine* e, int32_t n_seqs, int32_t t_max) {
   if (!e || n_seqs <= 0 || t_max <= 0) return -1;
+  if (e->lm) return lm_cache_bytes(e, n_seqs, t_max);
   return (int64_t)e->cfg.n_layers * 2 * n_seqs * e->cfg.d_model * (int64_t)t_max * 2;
 }
 
 extern "C" int arcb_session_create(arcb_engine* e, const arcb_session_desc* dsc, arcb_session** out) {
-  if (!e || !dsc || !out) return fail(ARCB_E_ARG, "null argument");
-  if (!engine_complete(e)) return fail(ARCB_E_STATE, "engine is missing tensors");
+  if (!e || !dsc || !out) return arcb_fail(ARCB_E_ARG, "null argument");
+  if (!engine_complete(e)) return arcb_fail(ARCB_E_STATE, "engine is missing tensors");
   if (dsc->n_seqs <= 0 || dsc->t_max <= 0 || dsc->max_new <= 0 || dsc->max_prefill_tokens <= 0)
-    return fail(ARCB_E_ARG, "bad session sizes");
-  if (!dsc->d_kv_cache || !dsc->d_workspace || !dsc->d_out_tokens) return fail(ARCB_E_ARG, "null buffer");
+    return arcb_fail(ARCB_E_ARG, "bad session sizes");
+  if (!dsc->d_kv_cache || !dsc->d_workspace || !dsc->d_out_tokens) return arcb_fail(ARCB_E_ARG, "null buffer");
   if (dsc->kv_cache_bytes < arcb_kv_cache_bytes(e, dsc->n_seqs, dsc->t_max))
-    return fail(ARCB_E_ARG, "kv cache too small");
+    return arcb_fail(ARCB_E_ARG, "kv cache too small");
   if (((uintptr_t)dsc->d_kv_cache & 255) || ((uintptr_t)dsc->d_workspace & 255))
-    return fail(ARCB_E_ARG, "buffers must be 256-byte aligned");
+    return arcb_fail(ARCB_E_ARG, "buffers must be 256-byte aligned");
+  if (e->lm) {
+    if (dsc->workspace_bytes < lm_workspace_bytes(e, dsc->n_seqs, dsc->max_prefill_tokens, dsc->attn_splits))
+      return arcb_fail(ARCB_E_ARG, "workspace too small");
+    arcb_session* s = new arcb_session();
+    s->eng = e;
+    s->desc = *dsc;
+    const int r = lm_session_create(s);
+    const cudaError_t ce = r ? cudaSuccess : cudaStreamCreateWithFlags(&s->capture_stream, cudaStreamNonBlocking);
+    if (r || ce != cudaSuccess) {
+      arcb_session_destroy(s);
+      return r ? r : arcb_fail_cuda(ce, "cudaStreamCreate");
+    }
+    *out = s;
+    return ARCB_OK;
+  }
   const int splits = choose_splits(e, dsc->n_seqs, dsc->attn_splits, dsc->t_max);
   const WsLayout w = ws_layout(e, dsc->n_seqs, dsc->max_prefill_tokens, choose_splits(e, dsc->n_seqs, dsc->attn_splits));
-  if ((size_t)dsc->workspace_bytes < w.total) return fail(ARCB_E_ARG, "workspace too small");
+  if ((size_t)dsc->workspace_bytes < w.total) return arcb_fail(ARCB_E_ARG, "workspace too small");
   arcb_session* s = new arcb_session();
   s->eng = e;
   s->desc = *dsc;
@@ -389,7 +328,7 @@ extern "C" int arcb_session_create(arcb_engine* e, const arcb_session_desc* dsc,
   s->state_ints = ints;
   s->n_state_ints = w.n_int;
   cudaError_t r = cudaStreamCreateWithFlags(&s->capture_stream, cudaStreamNonBlocking);
-  if (r != cudaSuccess) { delete s; return fail_cuda(r, "cudaStreamCreate"); }
+  if (r != cudaSuccess) { delete s; return arcb_fail_cuda(r, "cudaStreamCreate"); }
   if (cudaEventCreate(&s->probe_begin) != cudaSuccess || cudaEventCreate(&s->probe_end) != cudaSuccess) {
     cudaGetLastError();
     s->probe_begin = s->probe_end = nullptr;  // the probe is optional
@@ -400,6 +339,7 @@ extern "C" int arcb_session_create(arcb_engine* e, const arcb_session_desc* dsc,
 
 extern "C" int arcb_session_destroy(arcb_session* s) {
   if (!s) return ARCB_OK;
+  if (s->ls) lm_session_destroy(s->ls);
   if (s->graph_exec) cudaGraphExecDestroy(s->graph_exec);
   if (s->graph) cudaGraphDestroy(s->graph);
   if (s->capture_stream) cudaStreamDestroy(s->capture_stream);
@@ -505,16 +445,17 @@ static int run_layer(arcb_session* s, int l, int rows, const int* pos, const int
 }
 
 extern "C" int arcb_prefill(arcb_session* s, const arcb_prefill_args* a, void* stream_v) {
-  if (!s || !a) return fail(ARCB_E_ARG, "null argument");
+  if (!s || !a) return arcb_fail(ARCB_E_ARG, "null argument");
   if (a->n_tokens <= 0 || a->n_tokens > s->desc.max_prefill_tokens)
-    return fail(ARCB_E_ARG, "n_tokens outside (0, max_prefill_tokens]");
+    return arcb_fail(ARCB_E_ARG, "n_tokens outside (0, max_prefill_tokens]");
+  if (s->eng->lm) return lm_prefill(s, a, (cudaStream_t)stream_v);
   if (a->n_kv_rows < 0 || a->n_kv_rows > s->desc.max_prefill_tokens)
-    return fail(ARCB_E_ARG, "n_kv_rows outside [0, max_prefill_tokens]");
+    return arcb_fail(ARCB_E_ARG, "n_kv_rows outside [0, max_prefill_tokens]");
   if (!a->d_token_ids || !a->d_pos_xyz || !a->d_seq || !a->d_kv_slot || !a->d_kv_count)
-    return fail(ARCB_E_ARG, "null token arrays");
+    return arcb_fail(ARCB_E_ARG, "null token arrays");
   if (a->n_first < 0 || (a->n_first > 0 && (!a->d_first_row || !a->d_first_seq || !a->d_prompt_len ||
                                               !a->d_grid_x || !a->d_grid_y || !a->d_grid_in_output)))
-    return fail(ARCB_E_ARG, "null first-token arrays");
+    return arcb_fail(ARCB_E_ARG, "null first-token arrays");
   cudaStream_t stream = (cudaStream_t)stream_v;
   arcb_engine* e = s->eng;
   const arcb_config& c = e->cfg;
@@ -560,6 +501,7 @@ extern "C" int arcb_prefill(arcb_session* s, const arcb_prefill_args* a, void* s
 }
 
 static int record_decode_step(arcb_session* s, cudaStream_t stream) {
+  if (s->ls) return lm_record_step(s, stream);
   arcb_engine* e = s->eng;
   const arcb_config& c = e->cfg;
   const int B = s->desc.n_seqs;
@@ -582,8 +524,9 @@ static int record_decode_step(arcb_session* s, cudaStream_t stream) {
 }
 
 extern "C" int arcb_decode(arcb_session* s, int32_t n_steps, void* stream_v) {
-  if (!s) return fail(ARCB_E_ARG, "null session");
-  if (!s->armed) return fail(ARCB_E_STATE, "arcb_prefill with first-token rows must run before arcb_decode");
+  if (!s) return arcb_fail(ARCB_E_ARG, "null session");
+  if (!s->armed && !(s->ls && lm_armed(s)))
+    return arcb_fail(ARCB_E_STATE, "arcb_prefill with first-token rows must run before arcb_decode");
   if (n_steps <= 0) return ARCB_OK;
   cudaStream_t stream = (cudaStream_t)stream_v;
   for (int attempt = 0; !s->graph_exec && attempt < 2; ++attempt) {
@@ -608,7 +551,7 @@ extern "C" int arcb_decode(arcb_session* s, int32_t n_steps, void* stream_v) {
       continue;
     }
     if (r) return r;
-    return fail_cuda(ce, "capture / instantiate of the decode step");
+    return arcb_fail_cuda(ce, "capture / instantiate of the decode step");
   }
   for (int i = 0; i < n_steps; ++i) CK(cudaGraphLaunch(s->graph_exec, stream));
   arcb_count_launch(s->graph_kernels * n_steps);
@@ -616,10 +559,10 @@ extern "C" int arcb_decode(arcb_session* s, int32_t n_steps, void* stream_v) {
 }
 
 extern "C" int arcb_session_poll(arcb_session* s, int32_t* n_finished, int32_t* device_error, void* stream_v) {
-  if (!s) return fail(ARCB_E_ARG, "null session");
+  if (!s) return arcb_fail(ARCB_E_ARG, "null session");
   cudaStream_t stream = (cudaStream_t)stream_v;
   int nf = 0, err = 0;
-  CK(cudaMemcpyAsync(&nf, s->st.n_finished, 4, cudaMemcpyDeviceToHost, stream));
+  CK(cudaMemcpyAsync(&nf, s->ls ? lm_n_finished(s) : s->st.n_finished, 4, cudaMemcpyDeviceToHost, stream));
   CK(cudaMemcpyAsync(&err, s->eng->d_err, 4, cudaMemcpyDeviceToHost, stream));
   CK(cudaStreamSynchronize(stream));
   if (n_finished) *n_finished = nf;
@@ -628,13 +571,13 @@ extern "C" int arcb_session_poll(arcb_session* s, int32_t* n_finished, int32_t* 
     cudaMemsetAsync(s->eng->d_err, 0, 4, stream);
     char buf[96];
     snprintf(buf, sizeof buf, "device error word = %d", err);
-    return fail(ARCB_E_DEVICE, buf);
+    return arcb_fail(ARCB_E_DEVICE, buf);
   }
   return ARCB_OK;
 }
 
 extern "C" int arcb_engine_saturation_count(arcb_engine* e, int64_t* count, int32_t reset, void* stream_v) {
-  if (!e || !count) return fail(ARCB_E_ARG, "null argument");
+  if (!e || !count) return arcb_fail(ARCB_E_ARG, "null argument");
   cudaStream_t stream = (cudaStream_t)stream_v;
   int n = 0;
   CK(cudaMemcpyAsync(&n, e->d_err + 1, 4, cudaMemcpyDeviceToHost, stream));
@@ -645,13 +588,13 @@ extern "C" int arcb_engine_saturation_count(arcb_engine* e, int64_t* count, int3
 }
 
 extern "C" int arcb_session_attention_probe(arcb_session* s, float* ms) {
-  if (!s || !ms) return fail(ARCB_E_ARG, "null argument");
-  if (!s->probe_recorded || !s->graph_exec) return fail(ARCB_E_STATE, "no decode step has run yet");
+  if (!s || !ms) return arcb_fail(ARCB_E_ARG, "null argument");
+  if (!s->probe_recorded || !s->graph_exec) return arcb_fail(ARCB_E_STATE, "no decode step has run yet");
   cudaError_t r = cudaEventSynchronize(s->probe_end);
   if (r == cudaSuccess) r = cudaEventElapsedTime(ms, s->probe_begin, s->probe_end);
   if (r != cudaSuccess) {
     cudaGetLastError();  // a failed query must not be picked up by the next launch check
-    return fail_cuda(r, "attention probe");
+    return arcb_fail_cuda(r, "attention probe");
   }
   return ARCB_OK;
 }
@@ -661,7 +604,7 @@ extern "C" int arcb_session_attention_probe(arcb_session* s, float* ms) {
 // ---------------------------------------------------------------------------
 extern "C" int arcb_op_rmsnorm(const float* x, const float* w, void* out16, int32_t rows, int32_t d,
                                float eps, int32_t act_format, void* stream) {
-  if (!x || !w || !out16 || d % 4) return fail(ARCB_E_ARG, "bad rmsnorm arguments");
+  if (!x || !w || !out16 || d % 4) return arcb_fail(ARCB_E_ARG, "bad rmsnorm arguments");
   CKL(arcb_launch_rmsnorm(x, w, out16, rows, d, eps, act_format == ARCB_ACT_F16, (cudaStream_t)stream), "rmsnorm");
   return ARCB_OK;
 }
@@ -686,13 +629,13 @@ static int ensure_gemm_init() {
 
 extern "C" int arcb_op_gemm(const void* a16, const void* w, float* y, int32_t M, int32_t N, int32_t K,
                             int32_t act_format, int32_t gemm_path, void* stream) {
-  if (!a16 || !w || !y || M <= 0) return fail(ARCB_E_ARG, "bad gemm arguments");
+  if (!a16 || !w || !y || M <= 0) return arcb_fail(ARCB_E_ARG, "bad gemm arguments");
   CKL(ensure_gemm_init(), "gemm init");
-  if (N % 128 || K % 32) return fail(ARCB_E_ARG, "gemm needs N % 128 == 0 and K % 32 == 0");
+  if (N % 128 || K % 32) return arcb_fail(ARCB_E_ARG, "gemm needs N % 128 == 0 and K % 32 == 0");
   const int variant = gemm_path == ARCB_GEMM_TC_1CTA ? 1 : (gemm_path == ARCB_GEMM_TC_2CTA ? 2 : 0);
   bool tc = gemm_path == ARCB_GEMM_TC || variant != 0 || (gemm_path == ARCB_GEMM_AUTO);
   if (tc && !arcb_gemm_tc_supported(M, N, K)) {
-    if (gemm_path != ARCB_GEMM_AUTO) return fail(ARCB_E_ARG, "tcgen05 gemm needs K % 64 == 0");
+    if (gemm_path != ARCB_GEMM_AUTO) return arcb_fail(ARCB_E_ARG, "tcgen05 gemm needs K % 64 == 0");
     tc = false;
   }
   GemmEpilogue ep{};
@@ -703,13 +646,13 @@ extern "C" int arcb_op_gemm(const void* a16, const void* w, float* y, int32_t M,
 
 extern "C" int arcb_op_gemm_residual(const void* a16, const void* w, const float* bias, float* x, int32_t M,
                                      int32_t N, int32_t K, int32_t act_format, int32_t gemm_path, void* stream) {
-  if (!a16 || !w || !x || M <= 0) return fail(ARCB_E_ARG, "bad gemm arguments");
+  if (!a16 || !w || !x || M <= 0) return arcb_fail(ARCB_E_ARG, "bad gemm arguments");
   CKL(ensure_gemm_init(), "gemm init");
-  if (N % 128 || K % 32) return fail(ARCB_E_ARG, "gemm needs N % 128 == 0 and K % 32 == 0");
+  if (N % 128 || K % 32) return arcb_fail(ARCB_E_ARG, "gemm needs N % 128 == 0 and K % 32 == 0");
   const int variant = gemm_path == ARCB_GEMM_TC_1CTA ? 1 : (gemm_path == ARCB_GEMM_TC_2CTA ? 2 : 0);
   bool tc = gemm_path == ARCB_GEMM_TC || variant != 0 || (gemm_path == ARCB_GEMM_AUTO);
   if (tc && !arcb_gemm_tc_supported(M, N, K)) {
-    if (gemm_path != ARCB_GEMM_AUTO) return fail(ARCB_E_ARG, "tcgen05 gemm needs K % 64 == 0");
+    if (gemm_path != ARCB_GEMM_AUTO) return arcb_fail(ARCB_E_ARG, "tcgen05 gemm needs K % 64 == 0");
     tc = false;
   }
   GemmEpilogue ep{};
@@ -726,11 +669,11 @@ extern "C" int64_t arcb_gemm_splitk_scratch_bytes(int32_t M, int32_t N, int32_t 
 
 extern "C" int arcb_op_gemm_residual_splitk(const void* a16, const void* w, const float* bias, float* x, int32_t M,
                                             int32_t N, int32_t K, int32_t act_format, void* scratch, void* stream) {
-  if (!a16 || !w || !x || M <= 0) return fail(ARCB_E_ARG, "bad gemm arguments");
+  if (!a16 || !w || !x || M <= 0) return arcb_fail(ARCB_E_ARG, "bad gemm arguments");
   CKL(ensure_gemm_init(), "gemm init");
-  if (N % 128 || !arcb_gemm_tc_supported(M, N, K)) return fail(ARCB_E_ARG, "gemm needs N % 128 == 0 and K % 64 == 0");
+  if (N % 128 || !arcb_gemm_tc_supported(M, N, K)) return arcb_fail(ARCB_E_ARG, "gemm needs N % 128 == 0 and K % 64 == 0");
   if (!scratch || !arcb_gemm_splitk_bn(M, N, K))
-    return fail(ARCB_E_ARG, "the split-K kernel does not apply to this shape (arcb_gemm_splitk_scratch_bytes returned 0) or no scratch was given");
+    return arcb_fail(ARCB_E_ARG, "the split-K kernel does not apply to this shape (arcb_gemm_splitk_scratch_bytes returned 0) or no scratch was given");
   GemmEpilogue ep{};
   ep.mode = EPI_RESID; ep.M = M; ep.N = N; ep.x = x; ep.bias = bias; ep.splitk_scratch = reinterpret_cast<float*>(scratch);
   CKL(arcb_launch_gemm(a16, w, ep, K, act_format == ARCB_ACT_F16, true, (cudaStream_t)stream, 0), "gemm");
@@ -747,10 +690,10 @@ extern "C" int arcb_op_decode_attention(const void* q16, const void* k, const vo
                                         const uint8_t* item_skip, int32_t n_items, int32_t n_heads,
                                         int32_t t_max, int32_t n_splits, void* scratch, int32_t act_format,
                                         void* stream) {
-  if (!q16 || !k || !v || !out16 || !item_len) return fail(ARCB_E_ARG, "null attention argument");
+  if (!q16 || !k || !v || !out16 || !item_len) return arcb_fail(ARCB_E_ARG, "null attention argument");
   if (n_items <= 0 || n_heads <= 0 || t_max <= 0 || n_splits < 1 || n_splits > 64)
-    return fail(ARCB_E_ARG, "bad attention sizes");
-  if (n_splits > 1 && !scratch) return fail(ARCB_E_ARG, "split attention needs scratch");
+    return arcb_fail(ARCB_E_ARG, "bad attention sizes");
+  if (n_splits > 1 && !scratch) return arcb_fail(ARCB_E_ARG, "split attention needs scratch");
   AttnStreamArgs a{};
   a.q16 = q16; a.k = reinterpret_cast<const __nv_bfloat16*>(k); a.v = reinterpret_cast<const __nv_bfloat16*>(v);
   a.out16 = out16; a.item_seq = item_seq; a.item_len = item_len; a.item_skip = item_skip;
@@ -762,7 +705,7 @@ extern "C" int arcb_op_decode_attention(const void* q16, const void* k, const vo
 
 extern "C" int arcb_op_head(const float* x, const int32_t* row_index, const float* lnf_w, const float* lm_head,
                             float* logits, int32_t* argmax, int32_t rows, int32_t d, float eps, void* stream) {
-  if (!x || !lnf_w || !lm_head || d % 4) return fail(ARCB_E_ARG, "bad head arguments");
+  if (!x || !lnf_w || !lm_head || d % 4) return arcb_fail(ARCB_E_ARG, "bad head arguments");
   HeadArgs ha{};
   ha.mode = HEAD_PLAIN; ha.rows = rows; ha.d = d; ha.eps = eps; ha.x = x; ha.row_index = row_index;
   ha.lnf_w = lnf_w; ha.lm_head = lm_head; ha.logits = logits; ha.argmax = argmax;

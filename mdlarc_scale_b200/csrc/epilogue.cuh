@@ -9,7 +9,63 @@ enum : int {
   EPI_QKV_ROPE = 1,   // 3D RoPE on q,k; q -> q16, k/v -> KV cache    (src/inference.py:402-407)
   EPI_RESID = 2,      // x[m][n] += acc (+ bias[n])                   (src/inference.py:410-413)
   EPI_SWIGLU = 3,     // h16[m][j] = silu(g+bg) * (u+bu)              (src/transformer.py:446-449)
+  EPI_RELU2 = 4,      // out[m][n] = relu(acc)^2 in the activation format
+  EPI_HEADS = 5,      // fused mixer projection of a layered model (ProjArgs)
 };
+
+// Fused projection of a mixer: the output columns are sections of whole heads, every head padded to
+// 64, 128 or 256 columns (zero weights), every section starting at a multiple of 64 columns.
+// q, the recurrence's k and v, and the output gate land at their own columns of `out` [M][N];
+// attention keys and values go to the layer's cache rows; the recurrence's gates leave as fp32.
+struct ProjArgs {
+  int recurrent;         // 0 attention, 1 matrix-memory recurrence
+  int M, N;
+  int H, G;              // query heads, key/value heads
+  int dim, dimp, vdim, vdimp;
+  int off_q, off_k, off_v, off_g, off_gate;   // first column of each section, < 0: absent
+  const float* bias;     // [N] or null
+  const float* q_norm;   // [dimp] gains of the per-head RMS norm, null: no norm
+  const float* k_norm;
+  float eps, q_mul;      // q_mul: constant factor of the queries
+  float temp_coef;       // query gain 1 + coef ln(floor((p + 1) / every) + 1); every 0: none
+  int temp_every;
+  float gate_cap;
+  const int* pos;        // [M] position of the row (its cache slot), < 0: the row stores nothing
+  const int* seq;        // [M] cache row, null: row index
+  void* kcache;          // [n_seqs][G][t_max][dimp] in the activation format
+  void* vcache;          // [n_seqs][G][t_max][vdimp]
+  int t_max, n_seqs;
+  void* out;             // [M][N] activation format
+  float* gates;          // [M][2 H]: log input gates, then log forget gates
+  int fmt;
+  int* err;
+};
+
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + __expf(-x)); }
+__device__ __forceinline__ float sigmoid_exact(float x) { return 1.f / (1.f + expf(-x)); }
+
+// gain of a query at position p
+__device__ __forceinline__ float query_gain(const ProjArgs& a, int p) {
+  float g = a.q_mul;
+  if (a.temp_every > 0) g *= 1.f + a.temp_coef * logf((float)((p + 1) / a.temp_every) + 1.f);
+  return g;
+}
+// capped log gates of the recurrence from the biased pre-activation
+__device__ __forceinline__ float gate_log(float x, float cap, bool forget) {
+  const float z = cap * tanhf(x / cap);
+  if (!forget) return z;
+  return fminf(z, 0.f) - log1pf(expf(-fabsf(z)));   // log sigmoid
+}
+// cache row of (row m, key/value head 0), or -1 when the row stores nothing
+__device__ __forceinline__ long long proj_cache_row(const ProjArgs& a, int m) {
+  const int s = a.pos[m], b = a.seq ? a.seq[m] : m;
+  if (s < 0) return -1;
+  if (s >= a.t_max || b < 0 || b >= a.n_seqs) {
+    arcb_set_error(a.err, ARCB_DEV_BAD_INDEX);
+    return -1;
+  }
+  return (long long)b * a.G * a.t_max + s;
+}
 
 struct GemmEpilogue {
   int mode;
@@ -35,6 +91,7 @@ struct GemmEpilogue {
   const float* rope;  // cos_x | sin_x | cos_y | sin_y | cos_z | sin_z
   int max_x, max_y, max_z;
   int* err;           // error word; word 1 counts 16-bit saturations
+  ProjArgs pj;        // EPI_HEADS
 };
 
 struct RopeRow {
@@ -202,6 +259,14 @@ __device__ __forceinline__ void epi_resid_quad(const GemmEpilogue& e, int m, int
 
 __device__ __forceinline__ void epi_store_quad(const GemmEpilogue& e, int m, int n, float4 v) {
   *reinterpret_cast<float4*>(e.y + (size_t)m * e.N + n) = v;
+}
+
+__device__ __forceinline__ float relu2_f(float v) { v = fmaxf(v, 0.f); return v * v; }
+
+__device__ __forceinline__ void epi_relu2_quad(const GemmEpilogue& e, int m, int n, float4 v) {
+  v = make_float4(relu2_f(v.x), relu2_f(v.y), relu2_f(v.z), relu2_f(v.w));
+  if (e.act_f16 == 1 && fmaxf(fmaxf(v.x, v.y), fmaxf(v.z, v.w)) > 65504.f) arcb_count_saturation(e.err);
+  st_act4(e.out16, (size_t)m * e.N + n, v, e.act_f16);
 }
 
 __device__ __forceinline__ float silu_f(float g) { return __fdividef(g, 1.f + __expf(-g)); }

@@ -41,12 +41,12 @@ struct TcCfg {
 constexpr int EPI_STAGE_GROUP_BYTES = 128 * 32 * 4;
 template <int MODE>
 __host__ __device__ constexpr int epi_stage_bytes() {
-  return (MODE == EPI_RESID || MODE == EPI_SWIGLU || MODE == EPI_QKV_ROPE) ? 2 * EPI_STAGE_GROUP_BYTES : 0;
+  return (MODE == EPI_RESID || MODE == EPI_SWIGLU || MODE == EPI_QKV_ROPE || MODE == EPI_RELU2) ? 2 * EPI_STAGE_GROUP_BYTES : 0;
 }
 // epilogues that go through the staging buffers and the third tensor map
 template <int BN, int MODE>
 __host__ __device__ constexpr bool epi_staged() {
-  return MODE == EPI_RESID || ((MODE == EPI_SWIGLU || MODE == EPI_QKV_ROPE) && BN == 256);
+  return MODE == EPI_RESID || MODE == EPI_RELU2 || ((MODE == EPI_SWIGLU || MODE == EPI_QKV_ROPE) && BN == 256);
 }
 
 // Residual epilogue: x[m][n] += acc[m][n] (+ bias[n]) for this CTA's 128 rows and this group's
@@ -140,6 +140,44 @@ __device__ __forceinline__ void epilogue_swiglu_tma(const GemmEpilogue& ep, cons
   if (elected && m0 < ep.M) {
     tma_store_2d(tmap_h, stage_smem, (n_grp0 >> 7) * 64, m0);
     bulk_commit_group();
+  }
+}
+
+// relu(acc)^2 of this group's column half in the 16-bit activation format, 64 columns at a time through
+// the staging box and one bulk tensor store per box.
+template <int BN>
+__device__ __forceinline__ void epilogue_relu2_tma(const GemmEpilogue& ep, const CUtensorMap* tmap_h, uint32_t t_row,
+                                                   int m0, int n_tile0, int grp, int row_in_tile, uint32_t stage_smem,
+                                                   uint8_t* stage_ptr, bool elected) {
+  uint8_t* my_row = stage_ptr + row_in_tile * 128;
+  const int sw = row_in_tile & 7;
+#pragma unroll 1
+  for (int b = grp * (BN / 128); b < (grp + 1) * (BN / 128); ++b) {
+    const int n0 = n_tile0 + b * 64;
+    if (n0 >= ep.N) break;               // uniform over the group
+    if (elected) bulk_wait_read_all();   // the previous store has read the buffer
+    named_bar_sync(1 + grp, 128);
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      uint32_t r[32];
+      tmem_ld_32x32(t_row + b * 64 + half * 32, r);
+      tmem_wait_ld();
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        uint32_t w[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          w[i] = pack2_act_chk(relu2_f(__uint_as_float(r[8 * q + 2 * i])), relu2_f(__uint_as_float(r[8 * q + 2 * i + 1])),
+                               ep.act_f16, ep.err);
+        *reinterpret_cast<uint4*>(my_row + (((half * 4 + q) ^ sw) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
+      }
+    }
+    fence_proxy_async_smem();
+    named_bar_sync(1 + grp, 128);
+    if (elected && m0 < ep.M) {
+      tma_store_2d(tmap_h, stage_smem, n0, m0);
+      bulk_commit_group();
+    }
   }
 }
 
@@ -301,6 +339,7 @@ __device__ __forceinline__ void epilogue_tile(const GemmEpilogue& ep, uint32_t t
                                          __uint_as_float(r[4 * q + 2]), __uint_as_float(r[4 * q + 3]));
             const int n = n0 + 4 * q;
             if constexpr (MODE == EPI_RESID) epi_resid_quad(ep, m, n, v);
+            else if constexpr (MODE == EPI_RELU2) epi_relu2_quad(ep, m, n, v);
             else epi_store_quad(ep, m, n, v);
           }
         }
@@ -446,6 +485,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
       const uint32_t t_row = tmem_base + acc * BN + ((uint32_t)(quarter * 32) << 16);
       if constexpr (MODE == EPI_RESID)
         epilogue_resid_tma<BN>(ep, &tmap_x, t_row, m_blk * TC_BM, n_blk * BN, col_half, row_in_tile,
+                               base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
+                               base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
+      else if constexpr (MODE == EPI_RELU2)
+        epilogue_relu2_tma<BN>(ep, &tmap_x, t_row, m_blk * TC_BM, n_blk * BN, col_half, row_in_tile,
                                base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
                                base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
       else if constexpr (MODE == EPI_SWIGLU && BN == 256)
@@ -641,6 +684,10 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constan
       const uint32_t t_row = tmem_base + acc * BN + ((uint32_t)(quarter * 32) << 16);
       if constexpr (MODE == EPI_RESID)
         epilogue_resid_tma<BN>(ep, &tmap_x, t_row, m_blk * 256 + (int)rank * 128, n_blk * BN, col_half, row_in_tile,
+                               base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
+                               base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
+      else if constexpr (MODE == EPI_RELU2)
+        epilogue_relu2_tma<BN>(ep, &tmap_x, t_row, m_blk * 256 + (int)rank * 128, n_blk * BN, col_half, row_in_tile,
                                base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
                                base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
       else if constexpr (MODE == EPI_SWIGLU)
@@ -885,8 +932,8 @@ constexpr int SM_BM = 32, SM_BN = 128, SM_BK = 32;
 
 template <int MODE>
 __global__ void __launch_bounds__(256)
-gemm_simt_kernel(const uint16_t* __restrict__ A, const uint16_t* __restrict__ W, GemmEpilogue ep,
-                 int K, int a_f16) {
+gemm_simt_kernel(const void* __restrict__ Av, const void* __restrict__ Wv, GemmEpilogue ep,
+                 int K, int a_fmt) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float As[SM_BK][SM_BM + 1];
@@ -904,22 +951,31 @@ gemm_simt_kernel(const uint16_t* __restrict__ A, const uint16_t* __restrict__ W,
   const int w_n = tid >> 1, w_kh = (tid & 1) * 16;
   for (int k0 = 0; k0 < K; k0 += SM_BK) {
     {
-      uint2 raw = make_uint2(0u, 0u);
-      if (m0 + a_row < ep.M)
-        raw = *reinterpret_cast<const uint2*>(A + (size_t)(m0 + a_row) * K + k0 + a_kq);
-      const float2 f0 = unpack2_act(raw.x, a_f16), f1 = unpack2_act(raw.y, a_f16);
-      As[a_kq + 0][a_row] = f0.x;
-      As[a_kq + 1][a_row] = f0.y;
-      As[a_kq + 2][a_row] = f1.x;
-      As[a_kq + 3][a_row] = f1.y;
+      float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (m0 + a_row < ep.M) f = ld_act4(Av, (size_t)(m0 + a_row) * K + k0 + a_kq, a_fmt);
+      As[a_kq + 0][a_row] = f.x;
+      As[a_kq + 1][a_row] = f.y;
+      As[a_kq + 2][a_row] = f.z;
+      As[a_kq + 3][a_row] = f.w;
     }
-    {
+    if (a_fmt == 2) {
+      const float4* src = reinterpret_cast<const float4*>(reinterpret_cast<const float*>(Wv) + (size_t)(n0 + w_n) * K + k0 + w_kh);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float4 f = __ldg(src + j);
+        Ws[w_kh + 4 * j][w_n] = f.x;
+        Ws[w_kh + 4 * j + 1][w_n] = f.y;
+        Ws[w_kh + 4 * j + 2][w_n] = f.z;
+        Ws[w_kh + 4 * j + 3][w_n] = f.w;
+      }
+    } else {
+      const uint16_t* W = reinterpret_cast<const uint16_t*>(Wv);
       const uint4* src = reinterpret_cast<const uint4*>(W + (size_t)(n0 + w_n) * K + k0 + w_kh);
       const uint4 r0 = __ldg(src), r1 = __ldg(src + 1);
       const uint32_t w[8] = {r0.x, r0.y, r0.z, r0.w, r1.x, r1.y, r1.z, r1.w};
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
-        const float2 f = unpack2_act(w[j], a_f16);
+        const float2 f = unpack2_act(w[j], a_fmt);
         Ws[w_kh + 2 * j][w_n] = f.x;
         Ws[w_kh + 2 * j + 1][w_n] = f.y;
       }
@@ -953,6 +1009,9 @@ gemm_simt_kernel(const uint16_t* __restrict__ A, const uint16_t* __restrict__ W,
     } else if constexpr (MODE == EPI_RESID) {
       epi_resid_quad(ep, m, n, lo);
       epi_resid_quad(ep, m, n + 64, hi);
+    } else if constexpr (MODE == EPI_RELU2) {
+      epi_relu2_quad(ep, m, n, lo);
+      epi_relu2_quad(ep, m, n + 64, hi);
     } else {
       epi_store_quad(ep, m, n, lo);
       epi_store_quad(ep, m, n + 64, hi);
@@ -1052,7 +1111,9 @@ int arcb_gemm_init() {
   if ((e = set_tc_smem_attr<EPI_QKV_ROPE>()) != cudaSuccess) return (int)e;
   if ((e = set_tc_smem_attr<EPI_RESID>()) != cudaSuccess) return (int)e;
   if ((e = set_tc_smem_attr<EPI_SWIGLU>()) != cudaSuccess) return (int)e;
+  if ((e = set_tc_smem_attr<EPI_RELU2>()) != cudaSuccess) return (int)e;
   if ((e = set_tc2_smem_attr<EPI_STORE_F32>()) != cudaSuccess) return (int)e;
+  if ((e = set_tc2_smem_attr<EPI_RELU2>()) != cudaSuccess) return (int)e;
   if ((e = set_tc2_smem_attr<EPI_QKV_ROPE>()) != cudaSuccess) return (int)e;
   if ((e = set_tc2_smem_attr<EPI_RESID>()) != cudaSuccess) return (int)e;
   if ((e = set_tc2_smem_attr<EPI_SWIGLU>()) != cudaSuccess) return (int)e;
@@ -1178,6 +1239,9 @@ static int launch_gemm_mode(const void* a16, const void* w16, const GemmEpilogue
     if (MODE == EPI_RESID) {
       r = make_tmap_resid_f32(&tx, ep.x, (uint64_t)M, (uint64_t)N);
       if (r) return 1000 + r;
+    } else if (MODE == EPI_RELU2) {
+      r = arcb_make_tmap_2d_16b(&tx, ep.out16, (uint64_t)M, (uint64_t)N, 128, 64, act_f16);
+      if (r) return 1000 + r;
     } else if (MODE == EPI_SWIGLU && (pair || wide)) {
       // h16 [M][N / 2], 128 x 64 boxes (one accumulator group's outputs)
       r = arcb_make_tmap_2d_16b(&tx, ep.out16, (uint64_t)M, (uint64_t)(N / 2), 128, 64, act_f16);
@@ -1219,8 +1283,7 @@ static int launch_gemm_mode(const void* a16, const void* w16, const GemmEpilogue
   }
   dim3 grid(N / SM_BN, (M + SM_BM - 1) / SM_BM);
   const cudaError_t le = arcb_launch(gemm_simt_kernel<MODE>, grid, dim3(256), 0, stream,
-                                     reinterpret_cast<const uint16_t*>(a16), reinterpret_cast<const uint16_t*>(w16), ep,
-                                     K, act_f16);
+                                     a16, w16, ep, K, act_f16);
   arcb_count_launch(1);
   return (int)le;
 }
@@ -1230,12 +1293,13 @@ int arcb_launch_gemm(const void* a16, const void* w16, const GemmEpilogue& ep, i
   const int M = ep.M, N = ep.N;
   if (M <= 0) return 0;
   if (N % 128 != 0 || K % 32 != 0) return -1;
-  if (use_tc && !arcb_gemm_tc_supported(M, N, K)) return -1;
+  if (use_tc && (act_f16 == 2 || !arcb_gemm_tc_supported(M, N, K))) return -1;
   switch (ep.mode) {
     case EPI_STORE_F32: return launch_gemm_mode<EPI_STORE_F32>(a16, w16, ep, K, act_f16, use_tc, tc_variant, stream);
     case EPI_QKV_ROPE: return launch_gemm_mode<EPI_QKV_ROPE>(a16, w16, ep, K, act_f16, use_tc, tc_variant, stream);
     case EPI_RESID: return launch_gemm_mode<EPI_RESID>(a16, w16, ep, K, act_f16, use_tc, tc_variant, stream);
     case EPI_SWIGLU: return launch_gemm_mode<EPI_SWIGLU>(a16, w16, ep, K, act_f16, use_tc, tc_variant, stream);
+    case EPI_RELU2: return launch_gemm_mode<EPI_RELU2>(a16, w16, ep, K, act_f16, use_tc, tc_variant, stream);
   }
   return -1;
 }

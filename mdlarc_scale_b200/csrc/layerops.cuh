@@ -1,0 +1,72 @@
+// Row-wise kernels of layered models (embedding, norms, unfused projections, token picking) and their
+// argument blocks; see layerops.cu.
+#pragma once
+#include "epilogue.cuh"
+
+// Device-resident state of the decode loop of a layered session (arrays indexed by cache row).
+struct StepState {
+  int n_seqs, t_max, max_new, stop_on_end, end_token;
+  int* cur_len;        // positions cached
+  int* len0;           // cur_len when the sequence was armed
+  int* cur_tok;        // token the next step feeds
+  int* active;         // 1: the next step advances this sequence
+  int* pos;            // [B] position (= cache slot) of the fed token, -1: held (written by step_begin)
+  int* kv_len;         // [B] keys the step attends to, 0: held
+  int* finished;       // [B]
+  int* n_finished;
+  int* out_tokens;     // [B][max_new]
+  const int* forced;   // optional [B][max_new]
+  float* step_logits;  // optional [B][max_new][vocab]
+  float temperature;
+  int top_k;
+  unsigned long long sample_seed;
+  const int* sample_stream;
+  int* err;
+};
+
+struct LmEmbedArgs {
+  int rows, width, pitch, vocab, fmt;
+  const int* token_ids;    // [rows]; null in step_begin
+  const float* embed;      // [vocab][pitch]
+  float alpha;             // x leaves multiplied by the residual factor of the first sublayer
+  float* x;                // [rows][pitch]
+  void* xn;                // [rows][pitch] activation format
+};
+
+// y = norm(x) * w; xn gets y in the activation format, and x (optional) y * x_scale.
+struct LmNormArgs {
+  int kind;                // ARCB_NORM_*
+  int rows, width, pitch, fmt;
+  float eps, x_scale;
+  float* x;                // [.][pitch]
+  const float* w;          // [pitch]
+  void* xn;                // [rows][pitch]
+  int write_x;
+  const int* row_index;    // optional gather of rows of x (write_x 0)
+  float* dense;            // optional [rows][width]: y, without padding
+};
+
+enum : int { PICK_PLAIN = 0, PICK_FIRST = 1, PICK_DECODE = 2 };
+
+struct PickArgs {
+  int mode, rows, vocab, pitch;
+  float* logits;           // [rows][pitch] raw, scaled in place
+  float scale;
+  float* out;              // optional [rows][vocab]
+  const int* first_seq;    // PICK_FIRST
+  const int* prompt_len;
+};
+
+int arcb_launch_lm_embed(const LmEmbedArgs& a, cudaStream_t stream);
+int arcb_launch_step_begin(const StepState& st, const LmEmbedArgs& a, cudaStream_t stream);
+int arcb_launch_lm_norm(const LmNormArgs& a, cudaStream_t stream);
+int arcb_launch_proj_prep(const ProjArgs& a, const float* proj, cudaStream_t stream);
+int arcb_launch_pick(const PickArgs& a, const StepState& st, cudaStream_t stream);
+int arcb_launch_seg_commit(const StepState& st, const int* seg_seq, const int* seg_pos0, const int* seg_rows, int n,
+                           cudaStream_t stream);
+int arcb_launch_feed(const StepState& st, const int* seqs, const int* tokens, int n, cudaStream_t stream);
+// dst row = row_off + (r / rb) * rbp + r % rb, dst column = (c / cb) * cbp + c % cb, pitch dst_pitch;
+// container 0 = bfloat16, 1 = half holding the bf16-rounded value, 2 = fp32
+int arcb_launch_pack_blocks(const float* src, void* dst, long long rows, long long cols, int rb, int rbp, int row_off,
+                            int cb, int cbp, long long dst_pitch, int container, cudaStream_t stream);
+void arcb_count_launch(long long n);

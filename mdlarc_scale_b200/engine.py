@@ -82,15 +82,62 @@ def _cfg_get(cfg, name, default=None):
     return getattr(cfg, name, default)
 
 
-class Engine:
-    """Packed bf16 weights of one TinyTransformer on one B200 (``arcb_engine``)."""
+class EngineBase:
+    """Packed weights of one model on one B200 (``arcb_engine``): what every model family shares."""
 
-    def __init__(self, state_dict: dict, config, device="cuda:0", act_format: str = "f16",
-                 gemm_path: str = "auto", attn_path: str = "auto"):
+    vocab_size = VOCAB
+    end_token = END_TOKEN_ID
+    session_class: type            # set below: Session
+
+    def __init__(self, device):
         self.lib = _lib.load()
         self.device = torch.device(device)
         if self.device.type != "cuda":
             raise RuntimeError("the B200 engine needs a CUDA device; there is no CPU path")
+        self._handle = C.c_void_p()
+
+    def _load_id(self, kind_id: int, layer: int, t: torch.Tensor) -> None:
+        src = t.detach().to(device=self.device, dtype=torch.float32).contiguous()
+        _lib.check(self.lib.arcb_engine_load_tensor(self._handle, kind_id, layer, src.data_ptr(),
+                                                    src.numel(), _stream_ptr(self.device)))
+        torch.cuda.current_stream(self.device).synchronize()  # src may be a temporary
+
+    def close(self) -> None:
+        if getattr(self, "_handle", None) and self._handle.value:
+            self.lib.arcb_engine_destroy(self._handle)
+            self._handle = C.c_void_p()
+
+    def __del__(self):
+        try:
+            self.close()
+        except Exception:
+            pass
+
+    def saturation_count(self, reset: bool = True) -> int:
+        """Values clamped to the half range (or attention scores that overflowed it) since the last
+        reset: a warning that the model's activations do not fit IEEE half (use act_format="bf16")."""
+        n = C.c_int64(0)
+        with torch.cuda.device(self.device):
+            _lib.check(self.lib.arcb_engine_saturation_count(self._handle, C.byref(n), int(bool(reset)),
+                                                             _stream_ptr(self.device)))
+        return int(n.value)
+
+    def new_session(self, n_seqs: int, t_max: int, max_new: int, max_prefill_tokens: int,
+                    stop_on_end: bool = True, attn_splits: int = 0, forced: torch.Tensor | None = None,
+                    want_step_logits: bool = False, out_tokens: torch.Tensor | None = None,
+                    constraints: dict | None = None, temperature: float = 0.0, top_k: int = 0,
+                    sample_seed: int = 0, sample_stream=None, end_token: int | None = None) -> "Session":
+        return self.session_class(self, n_seqs, t_max, max_new, max_prefill_tokens, stop_on_end, attn_splits,
+                                  forced, want_step_logits, out_tokens, constraints, temperature, top_k,
+                                  sample_seed, sample_stream, self.end_token if end_token is None else end_token)
+
+
+class Engine(EngineBase):
+    """Packed bf16 weights of one TinyTransformer on one B200 (``arcb_engine``)."""
+
+    def __init__(self, state_dict: dict, config, device="cuda:0", act_format: str = "f16",
+                 gemm_path: str = "auto", attn_path: str = "auto"):
+        super().__init__(device)
         for name, want in (("rope_type", "3d"), ("norm_type", "rmsnorm"), ("ffn_type", "swiglu")):
             got = str(_cfg_get(config, name, want)).lower()
             if got != want:
@@ -115,7 +162,6 @@ class Engine:
             gemm_path={"auto": _lib.GEMM_AUTO, "simt": _lib.GEMM_SIMT, "tc": _lib.GEMM_TC}[gemm_path],
             attn_path={"auto": _lib.ATTN_AUTO, "stream": _lib.ATTN_STREAM}[attn_path],
             norm_eps=float(_cfg_get(config, "norm_eps", 1e-5)))
-        self._handle = C.c_void_p()
         with torch.cuda.device(self.device):
             _lib.check(self.lib.arcb_engine_create(C.byref(cfg), C.byref(self._handle)))
             tables = rope_tables(HEAD_DIM, cfg.max_x, cfg.max_y, cfg.max_z,
@@ -135,43 +181,11 @@ class Engine:
         return cls(model.state_dict(), model.config, device=device, **kw)
 
     def _load(self, kind: str, layer: int, t: torch.Tensor) -> None:
-        src = t.detach().to(device=self.device, dtype=torch.float32).contiguous()
-        _lib.check(self.lib.arcb_engine_load_tensor(self._handle, _lib.KIND[kind], layer, src.data_ptr(),
-                                                    src.numel(), _stream_ptr(self.device)))
-        torch.cuda.current_stream(self.device).synchronize()  # src may be a temporary
-
-    def close(self) -> None:
-        if getattr(self, "_handle", None) and self._handle.value:
-            self.lib.arcb_engine_destroy(self._handle)
-            self._handle = C.c_void_p()
-
-    def __del__(self):
-        try:
-            self.close()
-        except Exception:
-            pass
-
-    def saturation_count(self, reset: bool = True) -> int:
-        """Values clamped to the half range (or attention scores that overflowed it) since the last
-        reset: a warning that the model's activations do not fit IEEE half (use act_format="bf16")."""
-        n = C.c_int64(0)
-        with torch.cuda.device(self.device):
-            _lib.check(self.lib.arcb_engine_saturation_count(self._handle, C.byref(n), int(bool(reset)),
-                                                             _stream_ptr(self.device)))
-        return int(n.value)
+        self._load_id(_lib.KIND[kind], layer, t)
 
     # ------------------------------------------------------------------
     def kv_bytes_per_position(self) -> int:
         return self.n_layers * 2 * self.d_model * 2
-
-    def new_session(self, n_seqs: int, t_max: int, max_new: int, max_prefill_tokens: int,
-                    stop_on_end: bool = True, attn_splits: int = 0, forced: torch.Tensor | None = None,
-                    want_step_logits: bool = False, out_tokens: torch.Tensor | None = None,
-                    constraints: dict | None = None, temperature: float = 0.0, top_k: int = 0,
-                    sample_seed: int = 0, sample_stream=None) -> "Session":
-        return Session(self, n_seqs, t_max, max_new, max_prefill_tokens, stop_on_end, attn_splits,
-                       forced, want_step_logits, out_tokens, constraints, temperature, top_k, sample_seed,
-                       sample_stream)
 
 
 _ENGINES: "weakref.WeakKeyDictionary" = weakref.WeakKeyDictionary()
@@ -209,9 +223,9 @@ class Session:
     ``t_max`` is the capacity asked for; ``self.t_max`` is the row pitch the cache is laid out with
     (``cache_row_pitch``), which is what the library is given as its ``t_max``."""
 
-    def __init__(self, eng: Engine, n_seqs, t_max, max_new, max_prefill_tokens, stop_on_end,
+    def __init__(self, eng: EngineBase, n_seqs, t_max, max_new, max_prefill_tokens, stop_on_end,
                  attn_splits, forced, want_step_logits, out_tokens=None, constraints=None,
-                 temperature=0.0, top_k=0, sample_seed=0, sample_stream=None):
+                 temperature=0.0, top_k=0, sample_seed=0, sample_stream=None, end_token=END_TOKEN_ID):
         self.eng = eng
         self.n_seqs, self.t_max, self.max_new = int(n_seqs), cache_row_pitch(t_max), int(max_new)
         self.t_requested = int(t_max)
@@ -227,7 +241,7 @@ class Session:
         self.kv_cache = torch.empty(kv_bytes, dtype=torch.uint8, device=dev)
         self.workspace = torch.empty(ws_bytes, dtype=torch.uint8, device=dev)
         if out_tokens is None:
-            out_tokens = torch.full((self.n_seqs, self.max_new), END_TOKEN_ID, dtype=torch.int32, device=dev)
+            out_tokens = torch.full((self.n_seqs, self.max_new), end_token, dtype=torch.int32, device=dev)
         elif (out_tokens.dtype != torch.int32 or tuple(out_tokens.shape) != (self.n_seqs, self.max_new)
               or not out_tokens.is_contiguous() or out_tokens.device != dev):
             raise ValueError("out_tokens must be a contiguous int32 [n_seqs, max_new] tensor on the engine's device")
@@ -236,7 +250,7 @@ class Session:
         if forced is not None:
             self.forced = forced.to(device=dev, dtype=torch.int32).contiguous()
             assert self.forced.shape == (self.n_seqs, self.max_new)
-        self.step_logits = (torch.zeros((self.n_seqs, self.max_new, VOCAB), dtype=torch.float32, device=dev)
+        self.step_logits = (torch.zeros((self.n_seqs, self.max_new, eng.vocab_size), dtype=torch.float32, device=dev)
                             if want_step_logits else None)
         # soft decoding constraints: dict(palette_mask=[B,10] bool|None, target_shape=[B,2] int|None,
         # palette_penalty, shape_penalty, disallow_tokens)
@@ -273,7 +287,7 @@ class Session:
             d_palette_mask=_ptr(self.palette_mask), d_target_shape=_ptr(self.target_shape),
             palette_penalty=pal_pen, shape_penalty=shp_pen, disallow_token_mask=disallow,
             temperature=float(temperature), top_k=int(top_k or 0), sample_seed=int(sample_seed) & (2 ** 64 - 1),
-            d_sample_stream=_ptr(self.sample_stream))
+            d_sample_stream=_ptr(self.sample_stream), end_token=int(end_token))
         self._handle = C.c_void_p()
         with torch.cuda.device(dev):
             _lib.check(lib.arcb_session_create(eng._handle, C.byref(desc), C.byref(self._handle)))
@@ -327,6 +341,9 @@ class Session:
             _lib.check(self.eng.lib.arcb_session_poll(self._handle, C.byref(nf), C.byref(err),
                                                       _stream_ptr(self.eng.device)))
         return int(nf.value)
+
+
+EngineBase.session_class = Session
 
 
 # ---------------------------------------------------------------------------
