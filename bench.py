@@ -316,6 +316,157 @@ def profile_prefill(args):
                       "tflops": (lin + att) / t / 1e12, "frac_of_bf16_burst_peak": (lin + att) / t / 1e12 / 1672.1}))
 
 
+# Sizes of the layered-model benchmark: the closest existing model is a TinyTransformer of the same width and
+# depth (heads of 64, its feed-forward sized to the same number of weights).
+LAYERED_SIZES = {
+    "1280": dict(width=1280, heads=20, kv_heads=5, dim=64, vdim=64, ff=5120, tiny_ff=3456),
+    "2048": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, ff=8192, tiny_ff=5440),
+    "4096": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, ff=16384, tiny_ff=10944),
+}
+
+
+def layered_config(size: dict, n_layers: int, vocab: int = 32000) -> dict:
+    """Repeats [attention + feed-forward, mLSTM, attention on shared keys + feed-forward, mLSTM]."""
+    layers = []
+    for n in range(n_layers):
+        if n % 2:
+            layers.append({"type": "mlstm", "mlp": None,
+                           "mixer": {"heads": size["heads"], "dim": size["dim"], "vdim": size["vdim"], "gate_cap": 15.0}})
+            continue
+        m = {"heads": size["heads"], "kv_heads": size["kv_heads"], "dim": size["dim"], "vdim": size["vdim"],
+             "scale": size["dim"] ** -0.5, "q_temp": {"coef": 0.1, "every": 4096}}
+        if n % 4 == 2:
+            m["kv_from"] = n - 2
+        layers.append({"type": "attention", "mlp": {"kind": "dense", "ff": size["ff"]}, "mixer": m})
+    return {"architecture": "Vodavik", "width": size["width"], "vocab": vocab, "layers": layers, "norm": {"eps": 1e-6},
+            "postln_alpha": 2.0, "logit_scale": 1.0}
+
+
+def layered_engine(cfg: dict, dev, act_format: str = "f16"):
+    """Engine of seeded random weights, drawn on the device (nothing is computed with them on the host)."""
+    from mdlarc_scale_b200 import registry, vodavik
+    spec = vodavik.model_spec(cfg)
+    gen = torch.Generator(device=dev).manual_seed(0)
+    width, tensors = spec.width, {}
+    for (kind, n), name in vodavik.tensor_names(spec).items():
+        layer = spec.layers[n]
+        nkv = layer.kv_heads if layer.mixer == "attention" else layer.heads
+        shape = {"EMBED": (spec.vocab, width), "HEAD": (spec.vocab, width), "FINAL_NORM": (width,), "NORM1": (width,),
+                 "NORM2": (width,), "Q": (layer.heads * layer.dim, width), "Q_B": (layer.heads * layer.dim,),
+                 "K": (nkv * layer.dim, width), "K_B": (nkv * layer.dim,), "V": (nkv * layer.vdim, width),
+                 "V_B": (nkv * layer.vdim,), "G": (layer.heads * layer.vdim, width), "O": (width, layer.heads * layer.vdim),
+                 "Q_NORM": (layer.dim,), "K_NORM": (layer.dim,), "SINK": (layer.heads,),
+                 "HEAD_NORM": (layer.heads * layer.vdim,), "I": (layer.heads, width), "I_B": (layer.heads,),
+                 "F": (layer.heads, width), "F_B": (layer.heads,), "UP": (layer.d_ff, width), "DOWN": (width, layer.d_ff)}[kind]
+        std = 1.0 if kind == "EMBED" else shape[-1] ** -0.5 if len(shape) == 2 else 0.1
+        t = torch.randn(shape, generator=gen, device=dev) * std
+        if kind.endswith("NORM") or kind.startswith("NORM"):
+            t += 1.0
+        if kind == "F_B":
+            t += 4.0
+        tensors[name] = t
+    return registry.build_engine(cfg, tensors, dev, act_format)
+
+
+def bench_layered(args):
+    """Prefill and decode throughput of the Vodavik design (random weights) beside a TinyTransformer of equal
+    width and depth, same prompts and batch.  Device-timed with CUDA events; every pass streams far more than
+    the L2 cache holds."""
+    from mdlarc_scale_b200.engine import Engine, chunk_rows, plan_prefill
+    from mdlarc_scale_b200.layered import Segment
+    dev = torch.device("cuda", 0)
+    size = LAYERED_SIZES[args.layered]
+    n_layers, B, P, T = args.layered_layers, args.layered_batch, args.layered_prompts, args.layered_tokens
+    steps = args.layered_steps
+
+    def timed(fn, warm=3, reps=5):
+        for _ in range(warm):
+            fn()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize(dev)
+        e0.record()
+        for _ in range(reps):
+            fn()
+        e1.record()
+        torch.cuda.synchronize(dev)
+        return e0.elapsed_time(e1) / 1e3 / reps
+
+    out = {"benchmark": "layered models", "size": args.layered, "layers": n_layers, "prompts": P, "tokens": T,
+           "decode_batch": B, "decode_context": [T, T + steps], "data": "synthetic", "dtype": "bf16 weights, half operands"}
+    sampler = ClockSampler(0)
+    with sampler:
+        for which in args.layered_models.split(","):
+            if which == "vodavik":
+                eng = layered_engine(layered_config(size, n_layers), dev)
+                w = sum(s.heads * s.dim + s.heads * s.vdim * 2 + (0 if s.mixer == "attention" and s.kv_from >= 0 else
+                        s.kv_heads * (s.dim + s.vdim)) + 2 * s.d_ff for s in eng.spec.layers) * eng.spec.width
+                n_attn, heads, dd = sum(s.mixer == "attention" for s in eng.spec.layers), size["heads"], size["dim"] + size["vdim"]
+                sess = eng.new_session(P, T, 1, P * T, stop_on_end=False)
+                segs = [Segment(i, np.random.default_rng(i).integers(0, 32000, T).tolist()) for i in range(P)]
+
+                def prefill():
+                    sess.lens = [0] * P
+                    sess.prefill_segments(segs)
+            else:
+                cfg, sd = tiny_of_size(size, n_layers, T + steps + 8)
+                eng = Engine(sd, cfg, dev)
+                w = (4 * size["width"] + 3 * size["tiny_ff"]) * size["width"] * n_layers
+                n_attn, heads, dd = n_layers, size["width"] // 64, 128
+                sess = eng.new_session(P, T + 8, 8, P * T + 2 * P, stop_on_end=False)
+                ids = np.random.default_rng(0).integers(0, 10, (P, T))
+                plans = [plan_prefill(ids, np.zeros((P, T, 3), np.int64), np.ones((P, T), bool), r).to(dev)
+                         for r in chunk_rows(np.full(P, T), P * T + 2 * P)]
+
+                def prefill():
+                    for p in plans:
+                        sess.prefill(p, None)
+            t = timed(prefill)
+            sess.poll()
+            flop = P * T * 2.0 * w + P * n_attn * heads * dd * float(T) ** 2
+            r = {"prefill_tokens_per_s": P * T / t, "prefill_ms": t * 1e3, "prefill_tflops": flop / t / 1e12}
+            sess.close()
+            # decode: B sequences from a context of T, in prefill calls of bounded size
+            per = max(1, 65536 // T)
+            if which == "vodavik":
+                sess = eng.new_session(B, T + 4 * steps + 8, 4 * steps + 8, per * T, stop_on_end=False)
+                for b in range(0, B, per):
+                    sess.prefill_segments([Segment(i, segs[i % P].tokens, arm=True) for i in range(b, min(B, b + per))])
+            else:
+                sess = eng.new_session(B, T + 4 * steps + 8, 4 * steps + 8, per * T + 2 * per, stop_on_end=False)
+                ids = np.random.default_rng(0).integers(0, 10, (B, T))
+                for rows in chunk_rows(np.full(B, T), per * T + 2 * per):
+                    sess.prefill(plan_prefill(ids, np.zeros((B, T, 3), np.int64), np.ones((B, T), bool), rows).to(dev), None)
+            t = timed(lambda: sess.decode(steps), warm=1, reps=2) / steps
+            sess.poll()
+            r.update({"decode_ms_per_step": t * 1e3, "decode_tokens_per_s": B / t})
+            sess.close()
+            out[which] = r
+            del sess, eng
+            torch.cuda.empty_cache()
+    out["clocks"] = sampler.summary()
+    print(json.dumps(out))
+
+
+def tiny_of_size(size: dict, n_layers: int, max_seq_len: int):
+    """Configuration and seeded random weights of a TinyTransformer of the given width and depth."""
+    d, ff = size["width"], size["tiny_ff"]
+    cfg = dict(d_model=d, n_heads=d // 64, n_layers=n_layers, d_ff=ff, vocab_size=14, max_seq_len=max_seq_len, num_examples=8,
+               rope_type="3d", norm_type="rmsnorm", ffn_type="swiglu")
+    g = torch.Generator(device="cuda").manual_seed(0)
+
+    def mat(o, i):
+        return torch.randn(o, i, generator=g, device="cuda") * i ** -0.5
+    one, zero = (lambda n: torch.ones(n, device="cuda")), (lambda n: torch.zeros(n, device="cuda"))
+    sd = {"token_embed.weight": mat(14, d), "example_embed.weight": mat(8, d), "ln_f.weight": one(d), "lm_head.weight": mat(14, d)}
+    for n in range(n_layers):
+        sd.update({f"blocks.{n}.ln1.weight": one(d), f"blocks.{n}.ln2.weight": one(d),
+                   f"blocks.{n}.attn.qkv_proj.weight": mat(3 * d, d), f"blocks.{n}.attn.out_proj.weight": mat(d, d),
+                   f"blocks.{n}.ffn.fc_gate.weight": mat(ff, d), f"blocks.{n}.ffn.fc_gate.bias": zero(ff),
+                   f"blocks.{n}.ffn.fc_up.weight": mat(ff, d), f"blocks.{n}.ffn.fc_up.bias": zero(ff),
+                   f"blocks.{n}.ffn.fc_down.weight": mat(d, ff), f"blocks.{n}.ffn.fc_down.bias": zero(d)})
+    return cfg, sd
+
+
 def profile_long_context(args):
     """One wave of the prefill-heavy large configuration end to end: `--profile-long` prompts of 5
     pairs of 30x30 grids + a 30x30 test input (10 247 tokens each), then `--max-new` greedy tokens with
@@ -808,6 +959,15 @@ def main():
                     help="only run one wave of SEQS 10 247-token prompts + --max-new tokens (long-context decode)")
     ap.add_argument("--profile-decode-small", type=int, default=0, metavar="SEQS",
                     help="only run prefill + 15 decode steps of SEQS tiny prompts on a 64-position cache (ncu target)")
+    ap.add_argument("--layered", choices=sorted(LAYERED_SIZES), default=None,
+                    help="prefill and decode throughput of a layered model (Vodavik) of this width beside a TinyTransformer "
+                         "of equal width and depth, instead of the headline workload")
+    ap.add_argument("--layered-layers", type=int, default=8)
+    ap.add_argument("--layered-prompts", type=int, default=16, help="prompts of one prefill call")
+    ap.add_argument("--layered-tokens", type=int, default=2048, help="tokens per prompt and decode context")
+    ap.add_argument("--layered-batch", type=int, default=256, help="sequences of a decode step")
+    ap.add_argument("--layered-steps", type=int, default=64, help="decode steps per timed pass")
+    ap.add_argument("--layered-models", default="vodavik,tiny")
     ap.add_argument("--max-new", type=int, default=MAX_NEW,
                     help="tokens generated per sequence (the workload uses 931; smaller only for profiling)")
     args = ap.parse_args()
@@ -826,6 +986,9 @@ def main():
         return
     if not torch.cuda.is_available():
         raise SystemExit("bench.py needs a B200 GPU (the product path has no CPU fallback)")
+    if args.layered:
+        bench_layered(args)
+        return
     if args.profile_attn > 0:
         profile_attention(args)
         return

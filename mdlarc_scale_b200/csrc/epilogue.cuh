@@ -29,14 +29,13 @@ struct ProjArgs {
   float eps, q_mul;      // q_mul: constant factor of the queries
   float temp_coef;       // query gain 1 + coef ln(floor((p + 1) / every) + 1); every 0: none
   int temp_every;
-  float gate_cap;
   const int* pos;        // [M] position of the row (its cache slot), < 0: the row stores nothing
   const int* seq;        // [M] cache row, null: row index
   void* kcache;          // [n_seqs][G][t_max][dimp] in the activation format
   void* vcache;          // [n_seqs][G][t_max][vdimp]
   int t_max, n_seqs;
   void* out;             // [M][N] activation format
-  float* gates;          // [M][2 H]: log input gates, then log forget gates
+  float* gates;          // [M][2 H]: biased pre-activations of the input gates, then of the forget gates
   int fmt;
   int* err;
 };
@@ -49,12 +48,6 @@ __device__ __forceinline__ float query_gain(const ProjArgs& a, int p) {
   float g = a.q_mul;
   if (a.temp_every > 0) g *= 1.f + a.temp_coef * logf((float)((p + 1) / a.temp_every) + 1.f);
   return g;
-}
-// capped log gates of the recurrence from the biased pre-activation
-__device__ __forceinline__ float gate_log(float x, float cap, bool forget) {
-  const float z = cap * tanhf(x / cap);
-  if (!forget) return z;
-  return fminf(z, 0.f) - log1pf(expf(-fabsf(z)));   // log sigmoid
 }
 // cache row of (row m, key/value head 0), or -1 when the row stores nothing
 __device__ __forceinline__ long long proj_cache_row(const ProjArgs& a, int m) {

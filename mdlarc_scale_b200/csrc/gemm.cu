@@ -41,12 +41,13 @@ struct TcCfg {
 constexpr int EPI_STAGE_GROUP_BYTES = 128 * 32 * 4;
 template <int MODE>
 __host__ __device__ constexpr int epi_stage_bytes() {
-  return (MODE == EPI_RESID || MODE == EPI_SWIGLU || MODE == EPI_QKV_ROPE || MODE == EPI_RELU2) ? 2 * EPI_STAGE_GROUP_BYTES : 0;
+  return (MODE == EPI_RESID || MODE == EPI_SWIGLU || MODE == EPI_QKV_ROPE || MODE == EPI_RELU2 ||
+          MODE == EPI_HEADS) ? 2 * EPI_STAGE_GROUP_BYTES : 0;
 }
 // epilogues that go through the staging buffers and the third tensor map
 template <int BN, int MODE>
 __host__ __device__ constexpr bool epi_staged() {
-  return MODE == EPI_RESID || MODE == EPI_RELU2 || ((MODE == EPI_SWIGLU || MODE == EPI_QKV_ROPE) && BN == 256);
+  return MODE == EPI_RESID || MODE == EPI_RELU2 || MODE == EPI_HEADS || ((MODE == EPI_SWIGLU || MODE == EPI_QKV_ROPE) && BN == 256);
 }
 
 // Residual epilogue: x[m][n] += acc[m][n] (+ bias[n]) for this CTA's 128 rows and this group's
@@ -177,6 +178,123 @@ __device__ __forceinline__ void epilogue_relu2_tma(const GemmEpilogue& ep, const
     if (elected && m0 < ep.M) {
       tma_store_2d(tmap_h, stage_smem, n0, m0);
       bulk_commit_group();
+    }
+  }
+}
+
+// Fused mixer projection (ProjArgs), this group's column half of the tile, 64 columns at a time.  A 64-column
+// box lies inside one head of one section.  Heads with a norm take their sum of squares over the whole
+// head first (a 128-column head spans both groups of a 128-column tile: each reads all of it, tensor
+// memory is cheap to read twice), then the box is normed, scaled and stored.  Queries, output gates and
+// the recurrence's keys and values leave as staged 128 x 64 boxes; attention keys and values go to their
+// cache rows, 128 contiguous bytes per row; the recurrence's gate columns leave as fp32.
+template <int BN>
+__device__ __forceinline__ void epilogue_heads_tma(const GemmEpilogue& ep, const CUtensorMap* tmap_o, uint32_t t_row, int m0,
+                                                   int m, bool row_ok, int n_tile0, int grp, int row_in_tile,
+                                                   uint32_t stage_smem, uint8_t* stage_ptr, bool elected) {
+  const ProjArgs& p = ep.pj;
+  uint8_t* my_row = stage_ptr + row_in_tile * 128;
+  const int sw = row_in_tile & 7;
+  const int end_q = p.H * p.dimp;
+#pragma unroll 1
+  for (int b = grp * (BN / 128); b < (grp + 1) * (BN / 128); ++b) {
+    const int n0 = n_tile0 + b * 64;
+    if (n0 >= p.N) break;                // uniform over the group
+    if (p.off_gate >= 0 && n0 >= p.off_gate) {
+      // gate pre-activations (and the padding behind them)
+#pragma unroll 1
+      for (int half = 0; half < 2; ++half) {
+        const int j0 = n0 + half * 32 - p.off_gate;
+        if (j0 >= 2 * p.H) break;
+        uint32_t r[32];
+        tmem_ld_32x32(t_row + b * 64 + half * 32, r);
+        tmem_wait_ld();
+        if (row_ok) {
+          float* dst = p.gates + (size_t)m * 2 * p.H + j0;
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (j0 + i < 2 * p.H) dst[i] = __uint_as_float(r[i]) + (p.bias ? __ldg(p.bias + n0 + half * 32 + i) : 0.f);
+        }
+      }
+      continue;
+    }
+    const bool is_q = n0 < end_q;
+    const bool is_g = p.off_g >= 0 && n0 >= p.off_g;
+    const bool is_v = !is_g && p.off_v >= 0 && n0 >= p.off_v;
+    const bool is_k = !is_q && !is_g && !is_v && p.off_k >= 0;
+    if (!is_q && !is_g && !is_v && !is_k) continue;       // padding columns behind the last section
+    if (is_g && n0 >= p.off_g + p.H * p.vdimp) continue;
+    if (is_v && p.off_g < 0 && n0 >= p.off_v + p.G * p.vdimp) continue;
+    const float* gain = is_q ? p.q_norm : is_k ? p.k_norm : nullptr;
+    const int sec0 = is_q ? p.off_q : is_k ? p.off_k : is_v ? p.off_v : p.off_g;
+    const int width = (is_q || is_k) ? p.dimp : p.vdimp;
+    const int in_head = (n0 - sec0) & (width - 1);         // head widths are powers of two
+    float mul = 1.f;
+    if (gain) {
+      float ss = 0.f;
+#pragma unroll 1
+      for (int c = 0; c < width; c += 32) {
+        const int nn = n0 - in_head + c;
+        uint32_t r[32];
+        tmem_ld_32x32(t_row + (nn - n_tile0), r);
+        tmem_wait_ld();
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          const float v = __uint_as_float(r[i]) + (p.bias ? __ldg(p.bias + nn + i) : 0.f);
+          ss = fmaf(v, v, ss);
+        }
+      }
+      mul = 1.f / sqrtf(ss / (float)p.dim + p.eps);
+    }
+    const float post = is_q ? query_gain(p, row_ok && p.pos ? max(p.pos[m], 0) : 0) : 1.f;
+    const bool cached = !p.recurrent && (is_k || is_v);
+    uint16_t* crow = nullptr;
+    if (cached && row_ok) {
+      const long long cr = proj_cache_row(p, m);
+      if (cr >= 0)
+        crow = reinterpret_cast<uint16_t*>(is_k ? p.kcache : p.vcache) +
+               (size_t)(cr + (long long)((n0 - sec0) / width) * p.t_max) * width + in_head;
+    }
+    if (!cached) {
+      if (elected) bulk_wait_read_all();   // the previous store has read the buffer
+      named_bar_sync(1 + grp, 128);
+    }
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      uint32_t r[32];
+      tmem_ld_32x32(t_row + b * 64 + half * 32, r);
+      tmem_wait_ld();
+      const int nn = n0 + half * 32;
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        uint32_t w[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          float v[2];
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int c = q * 8 + i * 2 + e;
+            float t = __uint_as_float(r[c]);
+            if (p.bias) t += __ldg(p.bias + nn + c);
+            if (gain) t = (t * mul) * __ldg(gain + in_head + half * 32 + c);
+            t *= post;
+            if (is_g) t = sigmoid_f(t);
+            v[e] = t;
+          }
+          w[i] = pack2_act_chk(v[0], v[1], ep.act_f16, ep.err);
+        }
+        const uint4 w4 = make_uint4(w[0], w[1], w[2], w[3]);
+        if (!cached) *reinterpret_cast<uint4*>(my_row + (((half * 4 + q) ^ sw) << 4)) = w4;
+        else if (crow) *reinterpret_cast<uint4*>(crow + half * 32 + q * 8) = w4;
+      }
+    }
+    if (!cached) {
+      fence_proxy_async_smem();
+      named_bar_sync(1 + grp, 128);
+      if (elected && m0 < ep.M) {
+        tma_store_2d(tmap_o, stage_smem, n0, m0);
+        bulk_commit_group();
+      }
     }
   }
 }
@@ -487,6 +605,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
         epilogue_resid_tma<BN>(ep, &tmap_x, t_row, m_blk * TC_BM, n_blk * BN, col_half, row_in_tile,
                                base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
                                base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
+      else if constexpr (MODE == EPI_HEADS)
+        epilogue_heads_tma<BN>(ep, &tmap_x, t_row, m_blk * TC_BM, m, row_ok, n_blk * BN, col_half, row_in_tile,
+                               base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
+                               base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
       else if constexpr (MODE == EPI_RELU2)
         epilogue_relu2_tma<BN>(ep, &tmap_x, t_row, m_blk * TC_BM, n_blk * BN, col_half, row_in_tile,
                                base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
@@ -685,6 +807,10 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constan
       if constexpr (MODE == EPI_RESID)
         epilogue_resid_tma<BN>(ep, &tmap_x, t_row, m_blk * 256 + (int)rank * 128, n_blk * BN, col_half, row_in_tile,
                                base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
+                               base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
+      else if constexpr (MODE == EPI_HEADS)
+        epilogue_heads_tma<BN>(ep, &tmap_x, t_row, m_blk * 256 + (int)rank * 128, m, row_ok, n_blk * BN, col_half,
+                               row_in_tile, base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
                                base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
       else if constexpr (MODE == EPI_RELU2)
         epilogue_relu2_tma<BN>(ep, &tmap_x, t_row, m_blk * 256 + (int)rank * 128, n_blk * BN, col_half, row_in_tile,
@@ -1112,6 +1238,8 @@ int arcb_gemm_init() {
   if ((e = set_tc_smem_attr<EPI_RESID>()) != cudaSuccess) return (int)e;
   if ((e = set_tc_smem_attr<EPI_SWIGLU>()) != cudaSuccess) return (int)e;
   if ((e = set_tc_smem_attr<EPI_RELU2>()) != cudaSuccess) return (int)e;
+  if ((e = set_tc_smem_attr<EPI_HEADS>()) != cudaSuccess) return (int)e;
+  if ((e = set_tc2_smem_attr<EPI_HEADS>()) != cudaSuccess) return (int)e;
   if ((e = set_tc2_smem_attr<EPI_STORE_F32>()) != cudaSuccess) return (int)e;
   if ((e = set_tc2_smem_attr<EPI_RELU2>()) != cudaSuccess) return (int)e;
   if ((e = set_tc2_smem_attr<EPI_QKV_ROPE>()) != cudaSuccess) return (int)e;
@@ -1239,6 +1367,9 @@ static int launch_gemm_mode(const void* a16, const void* w16, const GemmEpilogue
     if (MODE == EPI_RESID) {
       r = make_tmap_resid_f32(&tx, ep.x, (uint64_t)M, (uint64_t)N);
       if (r) return 1000 + r;
+    } else if (MODE == EPI_HEADS) {
+      r = arcb_make_tmap_2d_16b(&tx, ep.pj.out, (uint64_t)M, (uint64_t)N, 128, 64, act_f16);
+      if (r) return 1000 + r;
     } else if (MODE == EPI_RELU2) {
       r = arcb_make_tmap_2d_16b(&tx, ep.out16, (uint64_t)M, (uint64_t)N, 128, 64, act_f16);
       if (r) return 1000 + r;
@@ -1299,6 +1430,9 @@ int arcb_launch_gemm(const void* a16, const void* w16, const GemmEpilogue& ep, i
     case EPI_QKV_ROPE: return launch_gemm_mode<EPI_QKV_ROPE>(a16, w16, ep, K, act_f16, use_tc, tc_variant, stream);
     case EPI_RESID: return launch_gemm_mode<EPI_RESID>(a16, w16, ep, K, act_f16, use_tc, tc_variant, stream);
     case EPI_SWIGLU: return launch_gemm_mode<EPI_SWIGLU>(a16, w16, ep, K, act_f16, use_tc, tc_variant, stream);
+    case EPI_HEADS:   // needs whole rows of a head in one thread: tensor-core kernels only
+      if (!use_tc) return -1;
+      return launch_gemm_mode<EPI_HEADS>(a16, w16, ep, K, act_f16, use_tc, tc_variant, stream);
     case EPI_RELU2: return launch_gemm_mode<EPI_RELU2>(a16, w16, ep, K, act_f16, use_tc, tc_variant, stream);
   }
   return -1;

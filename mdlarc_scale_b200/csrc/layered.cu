@@ -7,6 +7,7 @@
 #include <cstring>
 
 #include "attn_gqa.cuh"
+#include "attn_prefill_gqa.cuh"
 #include "engine.cuh"
 #include "gemm.cuh"
 #include "layerops.cuh"
@@ -76,7 +77,14 @@ struct LmWs {
   int head_rows;
 };
 
-bool use_fused(const LayeredModel& m) { return false && m.d.fused_proj; }
+// Head norms, gates and cache writes inside the projection product: the tensor-core kernels in a 16-bit
+// format, heads that fit a column tile.
+bool use_fused(const LayeredModel& m) {
+  if (m.fmt == 2 || m.d.gemm_path == ARCB_GEMM_SIMT || !m.d.fused_proj) return false;
+  for (const LmLayer& L : m.layers)
+    if (L.d.mixer == ARCB_MIXER_ATTENTION && L.d.qk_norm && L.dimp > 128) return false;
+  return true;
+}
 
 int lm_splits(const LayeredModel& m, int B, int requested, int t_max) {
   if (requested > 0) return requested > 64 ? 64 : requested;
@@ -160,6 +168,8 @@ extern "C" int arcb_engine_create_layered(const arcb_model_desc* md, const arcb_
   }
   if (!arcb_device_ok()) return arcb_fail(ARCB_E_UNSUPPORTED, "current device is not compute capability 10.x");
   CKL(arcb_gemm_init(), "gemm init (shared-memory opt-in / cuTensorMapEncodeTiled lookup)");
+  CKL(arcb_mlstm_chunk_init(), "chunkwise recurrence init (shared-memory opt-in)");
+  CKL(arcb_attn_prefill_gqa_init(), "prefill attention init (shared-memory opt-in)");
   arcb_engine* e = new arcb_engine();
   std::memset(&e->cfg, 0, sizeof e->cfg);
   cudaGetDevice(&e->device);
@@ -433,19 +443,23 @@ int lm_mixer(arcb_session* s, int l, const Rows& R, cudaStream_t stream) {
   p.eps = m.d.norm_eps;
   p.q_mul = rec ? 1.f / sqrtf((float)d.dim) : 1.f;
   p.temp_coef = d.q_temp_coef; p.temp_every = rec ? 0 : d.q_temp_every;
-  p.gate_cap = d.gate_cap;
   p.pos = R.pos; p.seq = R.seq; p.kcache = ls->k[l]; p.vcache = ls->v[l]; p.t_max = T; p.n_seqs = B;
   p.out = ls->proj; p.gates = ls->gates; p.fmt = m.fmt; p.err = s->eng->d_err;
   GemmEpilogue ep{};
   ep.M = R.n; ep.N = L.n_proj; ep.act_f16 = m.fmt; ep.err = s->eng->d_err;
-  ep.mode = EPI_STORE_F32; ep.y = ls->proj32;
-  CKL(lm_gemm(m, ls->xn, L.w_proj, ep, m.wp, stream), "projection gemm");
-  CKL(arcb_launch_proj_prep(p, ls->proj32, stream), "projection prep");
+  if (use_fused(m)) {
+    ep.mode = EPI_HEADS; ep.pj = p;
+    CKL(lm_gemm(m, ls->xn, L.w_proj, ep, m.wp, stream), "fused projection gemm");
+  } else {
+    ep.mode = EPI_STORE_F32; ep.y = ls->proj32;
+    CKL(lm_gemm(m, ls->xn, L.w_proj, ep, m.wp, stream), "projection gemm");
+    CKL(arcb_launch_proj_prep(p, ls->proj32, stream), "projection prep");
+  }
 
   if (rec) {
     MlstmArgs a{};
     a.proj = ls->proj; a.pitch = L.n_proj; a.off_q = L.off_q; a.off_k = L.off_k; a.off_v = L.off_v; a.off_g = L.off_g;
-    a.gates = ls->gates; a.norm_w = L.head_norm; a.out = ls->mix; a.S = ls->S[l]; a.n = ls->n[l]; a.m = ls->m[l];
+    a.gates = ls->gates; a.gate_cap = d.gate_cap; a.norm_w = L.head_norm; a.out = ls->mix; a.S = ls->S[l]; a.n = ls->n[l]; a.m = ls->m[l];
     a.H = d.heads; a.dim = d.dim; a.dimp = L.dimp; a.vdim = d.vdim; a.vdimp = L.vdimp; a.n_seqs = B; a.fmt = m.fmt;
     a.eps = m.d.norm_eps; a.err = s->eng->d_err;
     if (R.pa) {
@@ -454,7 +468,19 @@ int lm_mixer(arcb_session* s, int l, const Rows& R, cudaStream_t stream) {
     } else {
       a.pos = R.pos; a.n_segs = R.n;
     }
-    CKL(arcb_launch_mlstm_step(a, stream), "mlstm");
+    if (R.pa && m.d.mlstm_path == ARCB_MLSTM_AUTO && arcb_mlstm_chunk_supported(L.dimp, L.vdimp, m.fmt))
+      CKL(arcb_launch_mlstm_chunk(a, stream), "mlstm chunks");
+    else
+      CKL(arcb_launch_mlstm_step(a, stream), "mlstm");
+  } else if (R.pa && m.fmt != 2 && m.d.attn_path == ARCB_ATTN_AUTO && R.pa->n_qblocks > 0 &&
+             arcb_attn_prefill_gqa_supported(L.dimp, L.vdimp, B, d.kv_heads, T, d.scale)) {
+    AttnPrefillGqaArgs a{};
+    a.q = ls->proj; a.q_pitch = L.n_proj; a.q_col = L.off_q; a.k = ls->k[l]; a.v = ls->v[l];
+    if (L.off_g >= 0) { a.gate = reinterpret_cast<const uint8_t*>(ls->proj) + (size_t)L.off_g * m.es; a.gate_pitch = L.n_proj; }
+    a.out = ls->mix; a.seq = R.seq; a.kv_count = R.kv_len; a.qblock_row0 = R.pa->d_qblock_row0; a.qblock_rows = R.pa->d_qblock_rows;
+    a.sink = d.sink ? L.sink : nullptr; a.n_qblocks = R.pa->n_qblocks; a.n_rows = R.n; a.n_heads = d.heads; a.n_kv = d.kv_heads;
+    a.dimp = L.dimp; a.vdimp = L.vdimp; a.t_max = T; a.n_seqs = B; a.scale = d.scale; a.act_f16 = m.fmt; a.err = s->eng->d_err;
+    CKL(arcb_launch_attn_prefill_gqa(a, stream), "prefill attention");
   } else {
     AttnGqaArgs a{};
     const uint8_t* pr = reinterpret_cast<const uint8_t*>(ls->proj);
@@ -546,6 +572,7 @@ int lm_prefill(arcb_session* s, const arcb_prefill_args* a, cudaStream_t stream)
     return arcb_fail(ARCB_E_ARG, "null first-token arrays");
   if (a->n_logit_rows < 0 || (a->n_logit_rows > 0 && (!a->d_logit_row || !a->d_logits)))
     return arcb_fail(ARCB_E_ARG, "null logit arrays");
+  if (a->n_qblocks > 0 && (!a->d_qblock_row0 || !a->d_qblock_rows)) return arcb_fail(ARCB_E_ARG, "null query blocks");
   int r = lm_clear(s, stream);
   if (r) return r;
   CKL(arcb_launch_lm_embed(lm_embed_args(s, a->n_tokens, a->d_token_ids), stream), "embed");

@@ -170,10 +170,10 @@ proj_prep_kernel(ProjArgs a, const float* __restrict__ proj, int n_units) {
   else if (a.off_k >= 0 && u < 2 * nkv) { sec = V; h = u - nkv; }
   else { sec = LOGS; h = 0; }
 
-  if (sec == LOGS) {      // recurrence only: the log gates of all heads
+  if (sec == LOGS) {      // recurrence only: the gates of all heads
     for (int j = lane; j < 2 * a.H; j += 32) {
       const int c = a.off_gate + j;
-      a.gates[(size_t)m * 2 * a.H + j] = gate_log(row[c] + (a.bias ? a.bias[c] : 0.f), a.gate_cap, j >= a.H);
+      a.gates[(size_t)m * 2 * a.H + j] = row[c] + (a.bias ? a.bias[c] : 0.f);
     }
     return;
   }

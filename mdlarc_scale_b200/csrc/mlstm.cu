@@ -72,7 +72,8 @@ mlstm_step_kernel(MlstmArgs a) {
       s_k[tid] = tid < a.dim ? ld_act(a.proj, base + a.off_k + (size_t)h * a.dimp + tid, a.fmt) : 0.f;
     }
     const float4 v = ld_act4(a.proj, base + a.off_v + (size_t)h * VP + c4 * 4, a.fmt);
-    const float gi = a.gates[(size_t)row * 2 * a.H + h], gf = a.gates[(size_t)row * 2 * a.H + a.H + h];
+    const float gi = gate_log(a.gates[(size_t)row * 2 * a.H + h], a.gate_cap, false);
+    const float gf = gate_log(a.gates[(size_t)row * 2 * a.H + a.H + h], a.gate_cap, true);
     const float m_new = fmaxf(gf + m, gi);
     const float keep = expf(gf + m - m_new), add = expf(gi - m_new);
     m = m_new;

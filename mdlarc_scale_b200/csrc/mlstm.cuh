@@ -8,11 +8,19 @@
 #pragma once
 #include "common.cuh"
 
+// capped log gates of the recurrence from the biased pre-activation
+__device__ __forceinline__ float gate_log(float x, float cap, bool forget) {
+  const float z = cap * tanhf(x / cap);
+  if (!forget) return z;
+  return fminf(z, 0.f) - log1pf(expf(-fabsf(z)));   // log sigmoid
+}
+
 struct MlstmArgs {
   const void* proj;          // [rows][pitch] activation format: q, k, v and sigmoid output gates
   long long pitch;
   int off_q, off_k, off_v, off_g;
-  const float* gates;        // [rows][2 H] log input gates, then log forget gates
+  const float* gates;        // [rows][2 H] biased pre-activations of the input gates, then of the forget gates
+  float gate_cap;
   const float* norm_w;       // [H][vdimp]
   void* out;                 // [rows][H][vdimp] activation format
   float* S;                  // [n_seqs][H][dim][vdimp]
@@ -28,5 +36,8 @@ struct MlstmArgs {
   int* err;
 };
 
+bool arcb_mlstm_chunk_supported(int dimp, int vdimp, int fmt);
+int arcb_mlstm_chunk_init();
+int arcb_launch_mlstm_chunk(const MlstmArgs& a, cudaStream_t stream);
 int arcb_launch_mlstm_step(const MlstmArgs& a, cudaStream_t stream);
 void arcb_count_launch(long long n);
