@@ -15,6 +15,10 @@
 namespace {
 
 constexpr int GQA_WARPS = 4;
+#ifndef ARCB_GQA_STEPS
+#define ARCB_GQA_STEPS 4
+#endif
+constexpr int GQA_STEPS = ARCB_GQA_STEPS;   // most load steps in flight per warp and plane
 constexpr float GQA_LOG2E = 1.4426950408889634f;
 
 __host__ __device__ constexpr int gqa_max(int a, int b) { return a > b ? a : b; }
@@ -22,18 +26,38 @@ __host__ __device__ constexpr int gqa_min(int a, int b) { return a < b ? a : b; 
 // lanes that share one key: 16 bytes a lane of the wider of the two rows
 __host__ __device__ constexpr int gqa_lpr(int fmt, int dp, int vp) { return gqa_min(32, gqa_max(dp, vp) * (fmt == 2 ? 4 : 2) / 16); }
 
-// N consecutive elements -> fp32
+// two fp32 values in one 64-bit register pair, and the two-wide multiply-add on them
+__device__ __forceinline__ uint64_t f2_pack(float lo, float hi) {
+  uint64_t d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ float2 f2_unpack(uint64_t v) {
+  float2 f;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(v));
+  return f;
+}
+__device__ __forceinline__ uint64_t f2_fma(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t f2_mul(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+
+// 2 N consecutive elements -> N fp32 pairs
 template <int FMT, int N>
-__device__ __forceinline__ void gqa_unpack(const uint32_t* raw, float (&out)[N]) {
-  if constexpr (FMT == 2) {
+__device__ __forceinline__ void gqa_unpack(const uint32_t* raw, uint64_t (&out)[N]) {
 #pragma unroll
-    for (int i = 0; i < N; ++i) out[i] = __uint_as_float(raw[i]);
-  } else {
-#pragma unroll
-    for (int i = 0; i < N / 2; ++i) {
+  for (int i = 0; i < N; ++i) {
+    if constexpr (FMT == 2) {
+      out[i] = f2_pack(__uint_as_float(raw[2 * i]), __uint_as_float(raw[2 * i + 1]));
+    } else {
       const float2 f = unpack2_act(raw[i], FMT);
-      out[2 * i] = f.x;
-      out[2 * i + 1] = f.y;
+      out[i] = f2_pack(f.x, f.y);
     }
   }
 }
@@ -67,7 +91,7 @@ attn_gqa_kernel(AttnGqaArgs a) {
   constexpr int DE = DP / LPR, VE = VP / LPR;            // dims per lane
   constexpr int KW = DE * ES / 4, VW = VE * ES / 4;      // 32-bit words per lane and row
   constexpr int RPL = 32 / LPR;                          // rows per load step
-  constexpr int U = gqa_max(1, gqa_min(8, 32 / gqa_max(KW, VW)));   // load steps per iteration
+  constexpr int U = gqa_max(1, gqa_min(GQA_STEPS, 32 / gqa_max(KW, VW)));   // load steps per iteration
   constexpr int ROWS = U * RPL;
   constexpr int REC = VP + 4;
   __shared__ float s_part[GQA_WARPS][RT][REC];
@@ -98,25 +122,27 @@ attn_gqa_kernel(AttnGqaArgs a) {
 
   const int sub = lane / LPR, seg = lane % LPR;
   const int my_r = seg / (LPR / RT);                     // head whose scores this lane keeps
-  float q[RT][DE];
+  uint64_t q[RT][DE / 2];
 #pragma unroll
   for (int r = 0; r < RT; ++r) {
     const float sc = r < nh ? a.scale * GQA_LOG2E : 0.f;
     const int h = h0 + min(r, nh - 1);
 #pragma unroll
-    for (int e = 0; e < DE; ++e)
-      q[r][e] = ld_act(a.q, (size_t)item * a.q_pitch + (size_t)h * DP + seg * DE + e, FMT) * sc;
+    for (int e = 0; e < DE / 2; ++e) {
+      const size_t at = (size_t)item * a.q_pitch + (size_t)h * DP + seg * DE + 2 * e;
+      q[r][e] = f2_pack(ld_act(a.q, at, FMT) * sc, ld_act(a.q, at + 1, FMT) * sc);
+    }
   }
   const size_t row0 = ((size_t)seq * a.n_kv + g) * (size_t)a.t_max;
   const char* Kp = reinterpret_cast<const char*>(a.k) + (row0 * DP + seg * DE) * ES;
   const char* Vp = reinterpret_cast<const char*>(a.v) + (row0 * VP + seg * VE) * ES;
 
   float m = -INFINITY, l = 0.f;                          // of head my_r, this lane group's rows
-  float acc[RT][VE];
+  uint64_t acc[RT][VE / 2];
 #pragma unroll
   for (int r = 0; r < RT; ++r)
 #pragma unroll
-    for (int e = 0; e < VE; ++e) acc[r][e] = 0.f;
+    for (int e = 0; e < VE / 2; ++e) acc[r][e] = 0ull;
 
   for (int r0 = begin + wj * ROWS; r0 < end; r0 += ROWS * GQA_WARPS) {
     uint32_t kk[U][KW], vv[U][VW];
@@ -138,14 +164,16 @@ attn_gqa_kernel(AttnGqaArgs a) {
     float mx = m;
 #pragma unroll
     for (int u = 0; u < U; ++u) {
-      float kf[DE];
-      gqa_unpack<FMT, DE>(kk[u], kf);
+      uint64_t kf[DE / 2];
+      gqa_unpack<FMT, DE / 2>(kk[u], kf);
       float d[RT];
 #pragma unroll
       for (int r = 0; r < RT; ++r) {
-        d[r] = 0.f;
+        uint64_t d2 = f2_mul(q[r][0], kf[0]);
 #pragma unroll
-        for (int e = 0; e < DE; ++e) d[r] = fmaf(q[r][e], kf[e], d[r]);
+        for (int e = 1; e < DE / 2; ++e) d2 = f2_fma(q[r][e], kf[e], d2);
+        const float2 f = f2_unpack(d2);
+        d[r] = f.x + f.y;
       }
       // transposing butterfly: RT partial sums -> one complete sum per lane
 #pragma unroll
@@ -171,20 +199,22 @@ attn_gqa_kernel(AttnGqaArgs a) {
 #pragma unroll
     for (int r = 0; r < RT; ++r) {
       const float al = RT == 1 ? alpha : __shfl_sync(0xffffffffu, alpha, sub * LPR + r * (LPR / RT));
+      const uint64_t al2 = f2_pack(al, al);
 #pragma unroll
-      for (int e = 0; e < VE; ++e) acc[r][e] *= al;
+      for (int e = 0; e < VE / 2; ++e) acc[r][e] = f2_mul(acc[r][e], al2);
     }
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       const float p = exp2f(s[u] - m_safe);
       l += p;
-      float vf[VE];
-      gqa_unpack<FMT, VE>(vv[u], vf);
+      uint64_t vf[VE / 2];
+      gqa_unpack<FMT, VE / 2>(vv[u], vf);
 #pragma unroll
       for (int r = 0; r < RT; ++r) {
         const float pr = RT == 1 ? p : __shfl_sync(0xffffffffu, p, sub * LPR + r * (LPR / RT));
+        const uint64_t pr2 = f2_pack(pr, pr);
 #pragma unroll
-        for (int e = 0; e < VE; ++e) acc[r][e] = fmaf(pr, vf[e], acc[r][e]);
+        for (int e = 0; e < VE / 2; ++e) acc[r][e] = f2_fma(pr2, vf[e], acc[r][e]);
       }
     }
   }
@@ -204,9 +234,10 @@ attn_gqa_kernel(AttnGqaArgs a) {
       const int src = sub * LPR + r * (LPR / RT);
       const float ra = __shfl_sync(0xffffffffu, sa, src), rb = __shfl_sync(0xffffffffu, sb, src);
 #pragma unroll
-      for (int e = 0; e < VE; ++e) {
-        const float other = __shfl_xor_sync(0xffffffffu, acc[r][e], o);
-        acc[r][e] = acc[r][e] * ra + other * rb;
+      for (int e = 0; e < VE / 2; ++e) {
+        const float2 mine = f2_unpack(acc[r][e]);
+        const float ox = __shfl_xor_sync(0xffffffffu, mine.x, o), oy = __shfl_xor_sync(0xffffffffu, mine.y, o);
+        acc[r][e] = f2_pack(mine.x * ra + ox * rb, mine.y * ra + oy * rb);
       }
     }
   }
@@ -214,7 +245,8 @@ attn_gqa_kernel(AttnGqaArgs a) {
 #pragma unroll
     for (int r = 0; r < RT; ++r)
 #pragma unroll
-      for (int e = 0; e < VE; ++e) s_part[wj][r][seg * VE + e] = acc[r][e];
+      for (int e = 0; e < VE / 2; ++e)
+        *reinterpret_cast<float2*>(&s_part[wj][r][seg * VE + 2 * e]) = f2_unpack(acc[r][e]);
     if (seg % (LPR / RT) == 0) {
       s_part[wj][my_r][VP] = m;
       s_part[wj][my_r][VP + 1] = l;

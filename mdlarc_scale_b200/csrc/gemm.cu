@@ -196,6 +196,11 @@ __device__ __forceinline__ void epilogue_heads_tma(const GemmEpilogue& ep, const
   uint8_t* my_row = stage_ptr + row_in_tile * 128;
   const int sw = row_in_tile & 7;
   const int end_q = p.H * p.dimp;
+  // biases of whole heads exist in attention layers; the recurrence's bias vector only serves its gates
+  const float* bias = p.recurrent ? nullptr : p.bias;
+  const float gain_q = query_gain(p, row_ok && p.pos ? max(p.pos[m], 0) : 0);
+  int normed_head = -1;                  // first column of the head `mul` belongs to
+  float mul = 1.f;
 #pragma unroll 1
   for (int b = grp * (BN / 128); b < (grp + 1) * (BN / 128); ++b) {
     const int n0 = n_tile0 + b * 64;
@@ -229,24 +234,28 @@ __device__ __forceinline__ void epilogue_heads_tma(const GemmEpilogue& ep, const
     const int sec0 = is_q ? p.off_q : is_k ? p.off_k : is_v ? p.off_v : p.off_g;
     const int width = (is_q || is_k) ? p.dimp : p.vdimp;
     const int in_head = (n0 - sec0) & (width - 1);         // head widths are powers of two
-    float mul = 1.f;
-    if (gain) {
+    if (gain && normed_head != n0 - in_head) {
+      normed_head = n0 - in_head;
       float ss = 0.f;
 #pragma unroll 1
       for (int c = 0; c < width; c += 32) {
-        const int nn = n0 - in_head + c;
         uint32_t r[32];
-        tmem_ld_32x32(t_row + (nn - n_tile0), r);
+        tmem_ld_32x32(t_row + (normed_head + c - n_tile0), r);
         tmem_wait_ld();
 #pragma unroll
-        for (int i = 0; i < 32; ++i) {
-          const float v = __uint_as_float(r[i]) + (p.bias ? __ldg(p.bias + nn + i) : 0.f);
-          ss = fmaf(v, v, ss);
+        for (int q = 0; q < 8; ++q) {
+          float4 v = make_float4(__uint_as_float(r[4 * q]), __uint_as_float(r[4 * q + 1]), __uint_as_float(r[4 * q + 2]),
+                                 __uint_as_float(r[4 * q + 3]));
+          if (bias) {
+            const float4 bv = __ldg(reinterpret_cast<const float4*>(bias + normed_head + c) + q);
+            v.x += bv.x; v.y += bv.y; v.z += bv.z; v.w += bv.w;
+          }
+          ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
         }
       }
       mul = 1.f / sqrtf(ss / (float)p.dim + p.eps);
     }
-    const float post = is_q ? query_gain(p, row_ok && p.pos ? max(p.pos[m], 0) : 0) : 1.f;
+    const float post = (is_q ? gain_q : 1.f) * (gain ? mul : 1.f);
     const bool cached = !p.recurrent && (is_k || is_v);
     uint16_t* crow = nullptr;
     if (cached && row_ok) {
@@ -269,19 +278,24 @@ __device__ __forceinline__ void epilogue_heads_tma(const GemmEpilogue& ep, const
       for (int q = 0; q < 4; ++q) {
         uint32_t w[4];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          float v[2];
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            const int c = q * 8 + i * 2 + e;
-            float t = __uint_as_float(r[c]);
-            if (p.bias) t += __ldg(p.bias + nn + c);
-            if (gain) t = (t * mul) * __ldg(gain + in_head + half * 32 + c);
-            t *= post;
-            if (is_g) t = sigmoid_f(t);
-            v[e] = t;
+        for (int i = 0; i < 2; ++i) {
+          const int c = q * 8 + i * 4;
+          float4 v = make_float4(__uint_as_float(r[c]), __uint_as_float(r[c + 1]), __uint_as_float(r[c + 2]), __uint_as_float(r[c + 3]));
+          if (bias) {
+            const float4 bv = __ldg(reinterpret_cast<const float4*>(bias + nn + c));
+            v.x += bv.x; v.y += bv.y; v.z += bv.z; v.w += bv.w;
           }
-          w[i] = pack2_act_chk(v[0], v[1], ep.act_f16, ep.err);
+          if (is_g) {
+            v = make_float4(sigmoid_f(v.x), sigmoid_f(v.y), sigmoid_f(v.z), sigmoid_f(v.w));
+          } else {
+            v.x *= post; v.y *= post; v.z *= post; v.w *= post;
+            if (gain) {
+              const float4 gv = __ldg(reinterpret_cast<const float4*>(gain + in_head + half * 32 + c));
+              v.x *= gv.x; v.y *= gv.y; v.z *= gv.z; v.w *= gv.w;
+            }
+          }
+          w[2 * i] = pack2_act_chk(v.x, v.y, ep.act_f16, ep.err);
+          w[2 * i + 1] = pack2_act_chk(v.z, v.w, ep.act_f16, ep.err);
         }
         const uint4 w4 = make_uint4(w[0], w[1], w[2], w[3]);
         if (!cached) *reinterpret_cast<uint4*>(my_row + (((half * 4 + q) ^ sw) << 4)) = w4;

@@ -461,7 +461,7 @@ int lm_mixer(arcb_session* s, int l, const Rows& R, cudaStream_t stream) {
     a.proj = ls->proj; a.pitch = L.n_proj; a.off_q = L.off_q; a.off_k = L.off_k; a.off_v = L.off_v; a.off_g = L.off_g;
     a.gates = ls->gates; a.gate_cap = d.gate_cap; a.norm_w = L.head_norm; a.out = ls->mix; a.S = ls->S[l]; a.n = ls->n[l]; a.m = ls->m[l];
     a.H = d.heads; a.dim = d.dim; a.dimp = L.dimp; a.vdim = d.vdim; a.vdimp = L.vdimp; a.n_seqs = B; a.fmt = m.fmt;
-    a.eps = m.d.norm_eps; a.err = s->eng->d_err;
+    a.n_rows = R.n; a.eps = m.d.norm_eps; a.err = s->eng->d_err;
     if (R.pa) {
       a.seg_row0 = R.pa->d_seg_row0; a.seg_rows = R.pa->d_seg_rows; a.seg_seq = R.pa->d_seg_seq; a.seg_pos0 = R.pa->d_seg_pos0;
       a.n_segs = R.pa->n_segs;

@@ -233,7 +233,7 @@ proj_prep_kernel(ProjArgs a, const float* __restrict__ proj, int n_units) {
 }
 
 // ---- token picking: one CTA per row ----
-constexpr int PICK_THREADS = 256;
+constexpr int PICK_THREADS = 512;
 
 // Order-preserving map of a float to an unsigned key.
 __device__ __forceinline__ uint32_t float_key(float f) {
@@ -295,13 +295,20 @@ pick_kernel(PickArgs a, StepState st) {
   // scale, copy out, first maximum
   unsigned long long best = 0;
   float* step = (!bad && !held && in_range && st.step_logits) ? st.step_logits + ((size_t)b * st.max_new + out_idx) * a.vocab : nullptr;
-  for (int v = tid; v < a.vocab; v += PICK_THREADS) {
-    const float x = lg[v] * a.scale;
-    lg[v] = x;
-    if (a.out) a.out[(size_t)i * a.vocab + v] = x;
-    if (step) step[v] = x;
-    const unsigned long long key = ((unsigned long long)float_key(x) << 32) | (uint32_t)~v;
-    best = key > best ? key : best;
+  for (int v0 = tid * 4; v0 < a.vocab; v0 += PICK_THREADS * 4) {     // rows are padded to a multiple of 128
+    float4 f = *reinterpret_cast<const float4*>(lg + v0);
+    f.x *= a.scale; f.y *= a.scale; f.z *= a.scale; f.w *= a.scale;
+    *reinterpret_cast<float4*>(lg + v0) = f;
+    const float xs[4] = {f.x, f.y, f.z, f.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int v = v0 + e;
+      if (v >= a.vocab) break;
+      if (a.out) a.out[(size_t)i * a.vocab + v] = xs[e];
+      if (step) step[v] = xs[e];
+      const unsigned long long key = ((unsigned long long)float_key(xs[e]) << 32) | (uint32_t)~v;
+      best = key > best ? key : best;
+    }
   }
   if (a.mode == PICK_PLAIN || held) return;
   if (bad) { if (tid == 0) arcb_set_error(st.err, ARCB_DEV_BAD_INDEX); return; }

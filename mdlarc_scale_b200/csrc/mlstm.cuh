@@ -27,6 +27,7 @@ struct MlstmArgs {
   float* n;                  // [n_seqs][H][dimp]
   float* m;                  // [n_seqs][H]
   int H, dim, dimp, vdim, vdimp, n_seqs, fmt;
+  int n_rows;                // rows of proj
   float eps;
   // segments of consecutive rows; null seg_seq: row b belongs to sequence b (one row each) at position
   // pos[b], < 0 = held
