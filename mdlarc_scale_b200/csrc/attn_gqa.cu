@@ -38,10 +38,9 @@ int tiles_of(int rep) { return (rep + 3) / 4; }
 }  // namespace
 
 int arcb_attn_gqa_splits(int n_items, int n_kv, int rep, int t_max) {
-  // four-warp CTAs: aim for two waves of four on each of the 148 SMs (a wave and a bit would leave SMs idle at
-  // the end), with at least 128 cached rows per split
+  // four-warp CTAs: at least three for each of the 148 SMs, with at least 128 cached rows per split
   const long long work = (long long)n_items * n_kv * tiles_of(rep);
-  long long s = (148LL * 8 + work - 1) / work;
+  long long s = (148LL * 3 + work - 1) / work;
   if (t_max > 0 && s > t_max / 128) s = t_max / 128;
   if (s < 1) s = 1;
   if (s > 32) s = 32;

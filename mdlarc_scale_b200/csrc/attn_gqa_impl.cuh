@@ -4,7 +4,9 @@
 // split).  The warps take alternating slices of the cached prefix.  Inside a warp LPR lanes share one
 // key: each lane holds DE query dims of every query head of the tile and VE value dims of the
 // accumulators, so a key (value) row is loaded once, 16 bytes a lane, and used for all heads of the
-// tile.  Partial scores are reduced by a transposing butterfly: after it every lane holds the complete
+// tile.  Rows are copied asynchronously into a ring in shared memory several stages ahead; a lane reads back only
+// the bytes it copied itself, so the ring needs no barrier, and the bytes in flight cost no registers.
+// Partial scores are reduced by a transposing butterfly: after it every lane holds the complete
 // score of ONE head of the tile (head = (lane % LPR) / (LPR / RT)), so exponentials, maxima and sums
 // are computed once per (key, head) and the weights are handed back by shuffles.  Scores, weights and
 // sums are fp32.  Warps merge through shared memory in a fixed order.
@@ -15,10 +17,9 @@
 namespace {
 
 constexpr int GQA_WARPS = 4;
-#ifndef ARCB_GQA_STEPS
-#define ARCB_GQA_STEPS 4
+#ifndef ARCB_GQA_STAGES
+#define ARCB_GQA_STAGES 3
 #endif
-constexpr int GQA_STEPS = ARCB_GQA_STEPS;   // most load steps in flight per warp and plane
 constexpr float GQA_LOG2E = 1.4426950408889634f;
 
 __host__ __device__ constexpr int gqa_max(int a, int b) { return a > b ? a : b; }
@@ -62,39 +63,64 @@ __device__ __forceinline__ void gqa_unpack(const uint32_t* raw, uint64_t (&out)[
   }
 }
 
-// W 32-bit words from global memory (16- or 8-byte loads, no L1 allocation)
+// W 32-bit words, global -> shared, zeros when !valid
 template <int W>
-__device__ __forceinline__ void gqa_load(const void* p, uint32_t (&r)[W]) {
+__device__ __forceinline__ void gqa_copy(uint32_t dst, const void* src, bool valid) {
+  if constexpr (W % 4 == 0) {
+#pragma unroll
+    for (int i = 0; i < W / 4; ++i)
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + i * 512), "l"(reinterpret_cast<const char*>(src) + i * 16),
+                   "r"(valid ? 16 : 0) : "memory");
+  } else if constexpr (W == 2) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 8, %2;" ::"r"(dst), "l"(src), "r"(valid ? 8 : 0) : "memory");
+  } else {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(dst), "l"(src), "r"(valid ? 4 : 0) : "memory");
+  }
+}
+template <int W>
+__device__ __forceinline__ void gqa_fetch(const uint8_t* src, uint32_t (&r)[W]) {
   if constexpr (W % 4 == 0) {
 #pragma unroll
     for (int i = 0; i < W / 4; ++i) {
-      const uint4 t = ldg_stream16(reinterpret_cast<const uint4*>(p) + i);
+      const uint4 t = *reinterpret_cast<const uint4*>(src + i * 512);
       r[4 * i] = t.x; r[4 * i + 1] = t.y; r[4 * i + 2] = t.z; r[4 * i + 3] = t.w;
     }
+  } else if constexpr (W == 2) {
+    const uint2 t = *reinterpret_cast<const uint2*>(src);
+    r[0] = t.x; r[1] = t.y;
   } else {
-#pragma unroll
-    for (int i = 0; i < W / 2; ++i) {
-      const uint2 t = __ldg(reinterpret_cast<const uint2*>(p) + i);
-      r[2 * i] = t.x; r[2 * i + 1] = t.y;
-    }
-    if constexpr (W % 2) r[W - 1] = __ldg(reinterpret_cast<const uint32_t*>(p) + W - 1);
+    r[0] = *reinterpret_cast<const uint32_t*>(src);
   }
 }
+
+// Sizes of one instantiation.  A slot is what a warp loads of one plane in one step (its lanes' words side by
+// side, 16 bytes a lane at most); a stage is U slots of keys and U of values.
+template <int FMT, int DP, int VP>
+struct GqaCfg {
+  static constexpr int ES = FMT == 2 ? 4 : 2;
+  static constexpr int LPR = gqa_lpr(FMT, DP, VP);
+  static constexpr int DE = DP / LPR, VE = VP / LPR;            // dims per lane
+  static constexpr int KW = DE * ES / 4, VW = VE * ES / 4;      // 32-bit words per lane and row
+  static constexpr int RPL = 32 / LPR;                          // rows per load step
+  static constexpr int U = gqa_max(KW, VW) > 4 ? 2 : 4;         // load steps per stage
+  static constexpr int ROWS = U * RPL;
+  static constexpr int K_SLOT = 128 * KW, V_SLOT = 128 * VW;
+  static constexpr int STAGE = U * (K_SLOT + V_SLOT);
+  static constexpr int STAGES = ARCB_GQA_STAGES;
+  static constexpr int SMEM = GQA_WARPS * STAGES * STAGE;
+};
 
 template <int FMT, int DP, int VP, int RT>
 __global__ void __launch_bounds__(GQA_WARPS * 32)
 attn_gqa_kernel(AttnGqaArgs a) {
   pdl_launch_dependents();
   pdl_wait();
-  constexpr int ES = FMT == 2 ? 4 : 2;
-  constexpr int LPR = gqa_lpr(FMT, DP, VP);
-  constexpr int DE = DP / LPR, VE = VP / LPR;            // dims per lane
-  constexpr int KW = DE * ES / 4, VW = VE * ES / 4;      // 32-bit words per lane and row
-  constexpr int RPL = 32 / LPR;                          // rows per load step
-  constexpr int U = gqa_max(1, gqa_min(GQA_STEPS, 32 / gqa_max(KW, VW)));   // load steps per iteration
-  constexpr int ROWS = U * RPL;
+  using C = GqaCfg<FMT, DP, VP>;
+  constexpr int ES = C::ES, LPR = C::LPR, DE = C::DE, VE = C::VE, KW = C::KW, VW = C::VW, RPL = C::RPL, U = C::U, ROWS = C::ROWS;
   constexpr int REC = VP + 4;
-  __shared__ float s_part[GQA_WARPS][RT][REC];
+  static_assert(C::SMEM >= GQA_WARPS * RT * REC * 4, "the warps' partial results reuse the ring");
+  extern __shared__ __align__(16) uint8_t gqa_smem[];
+  float (*s_part)[RT][REC] = reinterpret_cast<float (*)[RT][REC]>(gqa_smem);
 
   const int lane = threadIdx.x & 31, wj = threadIdx.x >> 5;
   long long w = blockIdx.x;
@@ -144,28 +170,50 @@ attn_gqa_kernel(AttnGqaArgs a) {
 #pragma unroll
     for (int e = 0; e < VE / 2; ++e) acc[r][e] = 0ull;
 
-  for (int r0 = begin + wj * ROWS; r0 < end; r0 += ROWS * GQA_WARPS) {
-    uint32_t kk[U][KW], vv[U][VW];
+  uint8_t* ring = gqa_smem + wj * (C::STAGES * C::STAGE);
+  const uint32_t ring_addr = static_cast<uint32_t>(__cvta_generic_to_shared(ring));
+  constexpr int K_LANE = KW % 4 == 0 ? 16 : KW * 4, V_LANE = VW % 4 == 0 ? 16 : VW * 4;   // distance between lanes in a slot
+  auto issue = [&](int r0, int stage) {     // every lane commits, also past the end: the group count stays in step
+    const uint32_t st = ring_addr + stage * C::STAGE;
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       const int row = r0 + u * RPL + sub;
-#pragma unroll
-      for (int i = 0; i < KW; ++i) kk[u][i] = 0u;
-      if (row < end) gqa_load<KW>(Kp + (size_t)row * (DP * ES), kk[u]);
+      const bool ok = row < end;
+      gqa_copy<KW>(st + u * C::K_SLOT + lane * K_LANE, Kp + (size_t)(ok ? row : 0) * (DP * ES), ok);
     }
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       const int row = r0 + u * RPL + sub;
-#pragma unroll
-      for (int i = 0; i < VW; ++i) vv[u][i] = 0u;
-      if (row < end) gqa_load<VW>(Vp + (size_t)row * (VP * ES), vv[u]);
+      const bool ok = row < end;
+      gqa_copy<VW>(st + U * C::K_SLOT + u * C::V_SLOT + lane * V_LANE, Vp + (size_t)(ok ? row : 0) * (VP * ES), ok);
     }
+  };
+  constexpr int STEP = ROWS * GQA_WARPS;
+  int ahead = begin + wj * ROWS;            // first row of the next stage to issue
+  int put = 0, get = 0;
+#pragma unroll
+  for (int i = 0; i < C::STAGES - 1; ++i) {
+    if (ahead < end) issue(ahead, put);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    ahead += STEP;
+    ++put;
+  }
+  for (int r0 = begin + wj * ROWS; r0 < end; r0 += STEP) {
+    if (ahead < end) issue(ahead, put);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    ahead += STEP;
+    put = put + 1 == C::STAGES ? 0 : put + 1;
+    asm volatile("cp.async.wait_group %0;" ::"n"(C::STAGES - 1) : "memory");
+    const uint8_t* slot = ring + get * C::STAGE;
+    get = get + 1 == C::STAGES ? 0 : get + 1;
     float s[U];
     float mx = m;
 #pragma unroll
     for (int u = 0; u < U; ++u) {
+      uint32_t kw[KW];
+      gqa_fetch<KW>(slot + u * C::K_SLOT + lane * K_LANE, kw);
       uint64_t kf[DE / 2];
-      gqa_unpack<FMT, DE / 2>(kk[u], kf);
+      gqa_unpack<FMT, DE / 2>(kw, kf);
       float d[RT];
 #pragma unroll
       for (int r = 0; r < RT; ++r) {
@@ -196,19 +244,23 @@ attn_gqa_kernel(AttnGqaArgs a) {
     const float alpha = exp2f(m - m_safe);
     l *= alpha;
     m = mx;
+    if (__any_sync(0xffffffffu, alpha != 1.f)) {
 #pragma unroll
-    for (int r = 0; r < RT; ++r) {
-      const float al = RT == 1 ? alpha : __shfl_sync(0xffffffffu, alpha, sub * LPR + r * (LPR / RT));
-      const uint64_t al2 = f2_pack(al, al);
+      for (int r = 0; r < RT; ++r) {
+        const float al = RT == 1 ? alpha : __shfl_sync(0xffffffffu, alpha, sub * LPR + r * (LPR / RT));
+        const uint64_t al2 = f2_pack(al, al);
 #pragma unroll
-      for (int e = 0; e < VE / 2; ++e) acc[r][e] = f2_mul(acc[r][e], al2);
+        for (int e = 0; e < VE / 2; ++e) acc[r][e] = f2_mul(acc[r][e], al2);
+      }
     }
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       const float p = exp2f(s[u] - m_safe);
       l += p;
+      uint32_t vw[VW];
+      gqa_fetch<VW>(slot + U * C::K_SLOT + u * C::V_SLOT + lane * V_LANE, vw);
       uint64_t vf[VE / 2];
-      gqa_unpack<FMT, VE / 2>(vv[u], vf);
+      gqa_unpack<FMT, VE / 2>(vw, vf);
 #pragma unroll
       for (int r = 0; r < RT; ++r) {
         const float pr = RT == 1 ? p : __shfl_sync(0xffffffffu, p, sub * LPR + r * (LPR / RT));
@@ -241,6 +293,7 @@ attn_gqa_kernel(AttnGqaArgs a) {
       }
     }
   }
+  __syncthreads();     // every warp is done with its ring
   if (sub == 0) {
 #pragma unroll
     for (int r = 0; r < RT; ++r)
@@ -291,13 +344,22 @@ attn_gqa_kernel(AttnGqaArgs a) {
   }
 }
 
+template <int FMT, int DP, int VP, int RT>
+cudaError_t gqa_launch_one(const AttnGqaArgs& a, dim3 grid, cudaStream_t stream) {
+  using C = GqaCfg<FMT, DP, VP>;
+  if (C::SMEM > 48 * 1024) {
+    const cudaError_t e = cudaFuncSetAttribute(attn_gqa_kernel<FMT, DP, VP, RT>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM);
+    if (e != cudaSuccess) return e;
+  }
+  return arcb_launch(attn_gqa_kernel<FMT, DP, VP, RT>, grid, dim3(GQA_WARPS * 32), C::SMEM, stream, a);
+}
+
 template <int FMT, int DP, int VP>
 cudaError_t gqa_launch_dv(const AttnGqaArgs& a, dim3 grid, cudaStream_t stream) {
-  constexpr int LPR = gqa_lpr(FMT, DP, VP);
-  static_assert(LPR >= 4, "a key spans at least four lanes");
-  if (a.tile_rows == 1) return arcb_launch(attn_gqa_kernel<FMT, DP, VP, 1>, grid, dim3(GQA_WARPS * 32), 0, stream, a);
-  if (a.tile_rows == 2) return arcb_launch(attn_gqa_kernel<FMT, DP, VP, 2>, grid, dim3(GQA_WARPS * 32), 0, stream, a);
-  return arcb_launch(attn_gqa_kernel<FMT, DP, VP, 4>, grid, dim3(GQA_WARPS * 32), 0, stream, a);
+  static_assert(GqaCfg<FMT, DP, VP>::LPR >= 4, "a key spans at least four lanes");
+  if (a.tile_rows == 1) return gqa_launch_one<FMT, DP, VP, 1>(a, grid, stream);
+  if (a.tile_rows == 2) return gqa_launch_one<FMT, DP, VP, 2>(a, grid, stream);
+  return gqa_launch_one<FMT, DP, VP, 4>(a, grid, stream);
 }
 
 template <int FMT>
