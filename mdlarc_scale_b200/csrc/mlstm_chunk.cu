@@ -255,6 +255,11 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmap, MlstmArgs a) {
   }
   const int rt_s = warp & 3, kh = warp >> 2;  // score block of this warp: token rows, key half
   const float inv_v = 1.f / (float)a.vdim;
+  float2 gain[2];
+#pragma unroll
+  for (int nt = 0; nt < 2; ++nt)
+    gain[nt] = __ldg(reinterpret_cast<const float2*>(a.norm_w + (size_t)h * VP + warp * 16 + nt * 8 + 2 * t4));
+  uint16_t* out = reinterpret_cast<uint16_t*>(a.out) + ((size_t)row0 * a.H + h) * VP + warp * 16 + 2 * t4;
   chunk_barrier();
 
   for (int c = 0; c < n_chunks; ++c) {
@@ -389,7 +394,7 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmap, MlstmArgs a) {
       }
       float nq_lo = e_lo * f_qn[r_lo] + f_sum[r_lo], nq_hi = e_hi * f_qn[r_hi] + f_sum[r_hi];
       if (KH == 2) { nq_lo += f_sum[L + r_lo]; nq_hi += f_sum[L + r_hi]; }
-      const float d_lo = 1.f / (fmaxf(fabsf(nq_lo), f_em[r_lo]) + 1e-6f), d_hi = 1.f / (fmaxf(fabsf(nq_hi), f_em[r_hi]) + 1e-6f);
+      const float d_lo = __fdividef(1.f, fmaxf(fabsf(nq_lo), f_em[r_lo]) + 1e-6f), d_hi = __fdividef(1.f, fmaxf(fabsf(nq_hi), f_em[r_hi]) + 1e-6f);
       float s_lo = 0.f, s_hi = 0.f;
 #pragma unroll
       for (int nt = 0; nt < 2; ++nt) {
@@ -464,24 +469,28 @@ mlstm_chunk_kernel(const __grid_constant__ CUtensorMap tmap, MlstmArgs a) {
     }
     wait_for(bars + 16, c & 1);     // the output gates
     // ---- head norm, gain, output gate ----
+    float inv[L / 16][2];
+#pragma unroll
+    for (int rt = 0; rt < L / 16; ++rt)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        float ss = 0.f;
+#pragma unroll
+        for (int w = 0; w < NW; ++w) ss += f_ss[w * L + rt * 16 + g + e * 8];
+        inv[rt][e] = rsqrtf(ss * inv_v + a.eps);
+      }
 #pragma unroll
     for (int rt = 0; rt < L / 16; ++rt)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int r = rt * 16 + g + e * 8;
-        if (r >= n_tok) continue;
-        float ss = 0.f;
-#pragma unroll
-        for (int w = 0; w < NW; ++w) ss += f_ss[w * L + r];
-        const float inv = 1.f / sqrtf(ss * inv_v + a.eps);
-        const size_t row = (size_t)row0 + t0 + r;
+        uint16_t* dst = out + (size_t)(t0 + r) * (a.H * VP);
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt) {
-          const int v = warp * 16 + nt * 8 + 2 * t4;
-          const float2 gt = unpack2_act(*reinterpret_cast<const uint32_t*>(bp + buf * C::STAGE + tile_off(r, v >> 3) + (v & 7) * 2), F16 ? 1 : 0);
-          const float2 nw = __ldg(reinterpret_cast<const float2*>(a.norm_w + (size_t)h * VP + v));
-          const uint32_t o = pack2_act(acc[rt][nt][2 * e] * inv * nw.x * gt.x, acc[rt][nt][2 * e + 1] * inv * nw.y * gt.y, F16 ? 1 : 0);
-          *reinterpret_cast<uint32_t*>(reinterpret_cast<uint16_t*>(a.out) + (row * a.H + h) * VP + v) = o;
+          const float2 gt = unpack2_act(*reinterpret_cast<const uint32_t*>(bp + buf * C::STAGE + tile_off(r, warp * 2 + nt) + 4 * t4), F16 ? 1 : 0);
+          const uint32_t o = pack2_act(acc[rt][nt][2 * e] * inv[rt][e] * gain[nt].x * gt.x,
+                                       acc[rt][nt][2 * e + 1] * inv[rt][e] * gain[nt].y * gt.y, F16 ? 1 : 0);
+          if (r < n_tok) *reinterpret_cast<uint32_t*>(dst + nt * 8) = o;
         }
       }
     chunk_barrier();     // n is updated; the tiles and the gates' buffer are free
