@@ -9,6 +9,8 @@ for the full 931-token budget over a static KV cache of 1536 positions.  One ste
 the hot path over one such batch: packed prefill + 930 graph-replayed decode steps.  Under
 torchrun every rank runs its own batch (weak scaling, no data-path collective).
 
+`--layered 1280|2048|4096` measures a layered model (Vodavik) beside a TinyTransformer of equal size instead.
+
 Prints ONE JSON line (rank 0): generated tokens/s over all GPUs, device-timed (`value`, inputs
 resident in HBM) and end to end through `generate_output` from pinned host tensors (`e2e`),
 plus the roofline of the dominant kernel (decode attention, HBM-bound), the CPU baseline, clocks.
