@@ -128,18 +128,28 @@ int arcb_engine_saturation_count(arcb_engine* eng, int64_t* count, int32_t reset
 
 #define ARCB_MIXER_ATTENTION 0 /* causal softmax attention, H query heads on G key/value heads          */
 #define ARCB_MIXER_MLSTM 1     /* matrix memory with exponential input gate and stabiliser (mLSTM)      */
+#define ARCB_MIXER_LATENT 2    /* softmax attention over a cached latent and one rotated key part       */
 
 #define ARCB_MLP_NONE 0
 #define ARCB_MLP_RELU2 1       /* W_down relu(W_up x)^2                                                 */
+#define ARCB_MLP_GLU 2         /* W_down glu(W_gate x, W_up x)                                          */
+#define ARCB_MLP_MOE 3         /* routed experts of the GLU form, and a shared one                      */
+
+#define ARCB_GLU_SILU 0        /* g sigmoid(g) u                                                        */
+#define ARCB_GLU_CLAMPED 1     /* g <= limit, |u| <= limit: g sigmoid(1.702 g) (u + 1)                  */
 
 #define ARCB_NORM_RMS 0
 #define ARCB_NORM_LAYER 1      /* centred, gain only                                                    */
+
+#define ARCB_PLACE_POST 0      /* x <- norm1(alpha x + mixer(x)), x <- norm2(alpha x + mlp(x))          */
+#define ARCB_PLACE_SANDWICH 1  /* x <- x + norm1b(mixer(norm1(x))), x <- x + norm2b(mlp(norm2(x)))      */
 
 typedef struct arcb_layer_desc {
   int32_t mixer;        /* ARCB_MIXER_*                                                                 */
   int32_t heads;        /* query heads (attention) / memory heads (mLSTM)                               */
   int32_t kv_heads;     /* attention: key/value heads, divides heads                                    */
-  int32_t dim, vdim;    /* per-head query/key and value size, 1..256                                    */
+  int32_t dim, vdim;    /* per-head query/key and value size, 1..256 (latent: dim counts the unrotated
+                         * query/key dimensions, any size)                                              */
   int32_t kv_from;      /* attention: layer whose cached keys and values are read, -1 = its own         */
   int32_t qkv_bias;     /* projections of q, k and v have biases                                        */
   int32_t qk_norm;      /* per-head RMS norm of queries and keys                                        */
@@ -150,12 +160,27 @@ typedef struct arcb_layer_desc {
   int32_t q_temp_every;
   float gate_cap;       /* mLSTM: gates are cap * tanh(. / cap)                                         */
   int32_t mlp;          /* ARCB_MLP_*                                                                   */
-  int32_t d_ff;
+  int32_t d_ff;         /* hidden size (ARCB_MLP_MOE: of one expert)                                    */
+  int32_t window;       /* both attentions: position i sees [i - window + 1, i], 0 = every earlier one  */
+  int32_t q_rank;       /* latent: size of the query latent, of the cached latent, of the rotated key   */
+  int32_t kv_rank;
+  int32_t rot_dim;
+  int32_t rot_dims;     /* leading dimensions of the rotated part that turn, in neighbouring pairs      */
+  double rot_base;      /* pair i turns by position * base^(-2 i / rot_dims)                            */
+  int32_t glu;          /* ARCB_GLU_* of the feed-forward, of the experts and of the shared expert      */
+  float glu_limit;      /* clamp of the feed-forward or of the experts                                  */
+  int32_t experts, top; /* ARCB_MLP_MOE: the `top` largest of sigmoid(W_router x); each chosen score    *
+                         * multiplies its expert's input                                                */
+  int32_t shared_ff;    /* hidden size of the expert every token passes, 0 = none                       */
+  float shared_limit;
 } arcb_layer_desc;
 
-/* Norms sit AFTER the residual sum: x <- norm1(alpha x + mixer(x)), x <- norm2(alpha x + mlp(x)). */
+/* Layers loop_start .. loop_stop - 1 run loop_times times in a row with the same weights, every pass on a
+ * cache of its own; the embedding is added to x ahead of every pass but the first.  loop_times 1 = no loop. */
 typedef struct arcb_model_desc {
   int32_t width, vocab, n_layers;
+  int32_t norm_place;   /* ARCB_PLACE_*                                                                 */
+  int32_t loop_start, loop_stop, loop_times;
   int32_t norm;         /* ARCB_NORM_*, all norms of the residual stream                                */
   int32_t act_format;   /* ARCB_ACT_*                                                                   */
   int32_t gemm_path;    /* ARCB_GEMM_AUTO / ARCB_GEMM_SIMT                                              */
@@ -192,6 +217,23 @@ enum arcb_lm_tensor_kind {
   ARCB_L_F_B,
   ARCB_L_UP,          /* [d_ff, width]                                   */
   ARCB_L_DOWN,        /* [width, d_ff]                                   */
+  ARCB_L_NORM1B,      /* [width], sandwich norms                         */
+  ARCB_L_NORM2B,
+  ARCB_L_DQ,          /* [q_rank, width]                                 */
+  ARCB_L_DQ_NORM,     /* [q_rank]                                        */
+  ARCB_L_UQ,          /* [heads * (dim + rot_dim), q_rank]               */
+  ARCB_L_DKV,         /* [kv_rank + rot_dim, width]                      */
+  ARCB_L_DKV_NORM,    /* [kv_rank]                                       */
+  ARCB_L_UK,          /* [heads * dim, kv_rank]                          */
+  ARCB_L_UV,          /* [heads * vdim, kv_rank]                         */
+  ARCB_L_GATE,        /* [d_ff, width]                                   */
+  ARCB_L_ROUTER,      /* [experts, width]                                */
+  ARCB_L_EXPERT_GATE, /* [experts, d_ff, width]                          */
+  ARCB_L_EXPERT_UP,
+  ARCB_L_EXPERT_DOWN, /* [experts, width, d_ff]                          */
+  ARCB_L_SHARED_GATE, /* [shared_ff, width]                              */
+  ARCB_L_SHARED_UP,
+  ARCB_L_SHARED_DOWN, /* [width, shared_ff]                              */
   ARCB_L_COUNT
 };
 
@@ -311,8 +353,23 @@ typedef struct arcb_prefill_args {
   int32_t n_logit_rows;        /* rows whose logits are wanted without arming the decode loop */
   const int32_t* d_logit_row;  /* [n_logit_rows]                               */
   float* d_logits;             /* [n_logit_rows][vocab]                        */
-  float* d_residuals;          /* optional [n_layers][n_tokens][width]: residual stream after every layer */
+  float* d_residuals;          /* optional [n_layer_runs][n_tokens][width]: residual stream after every layer run */
+  /* Latent attention on the tensor cores: the keys and values of the call's query blocks are expanded from the
+   * cached latents into a scratch of arcb_session_expand_rows rows, group by group.  Group g covers the query
+   * blocks [h_group_qblock[g], h_group_qblock[g + 1]) and the 128-row scratch tiles [h_group_tile[g],
+   * h_group_tile[g + 1]), which start at scratch row 0 again in every group.  d_tile_src: latent row (cache row *
+   * t_max + position) of each tile's first row.  d_qblock_kv0 (above): scratch row, within the block's group, that
+   * position 0 of the block's sequence would have (may be negative); it must cover every key the window leaves
+   * visible.  Optional: without groups the streaming kernel runs. */
+  int32_t n_groups;
+  const int32_t* h_group_qblock; /* host, [n_groups + 1] */
+  const int32_t* h_group_tile;   /* host, [n_groups + 1] */
+  const int32_t* d_tile_src;
 } arcb_prefill_args;
+
+/* Layered engines: rows of the session's expansion scratch (0: no layer uses it) and the widest window of the
+ * layers that do (t_max when one sees everything). */
+int arcb_session_expand_rows(arcb_session* s, int32_t* rows, int32_t* window);
 
 int arcb_prefill(arcb_session* s, const arcb_prefill_args* a, void* stream);
 

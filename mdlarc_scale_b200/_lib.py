@@ -25,12 +25,16 @@ KIND = {name: i for i, name in enumerate(TENSOR_KINDS)}
 # layered engines (enum arcb_lm_tensor_kind and the mixer / feed-forward / norm codes)
 LAYERED_KINDS = [
     "EMBED", "FINAL_NORM", "HEAD", "NORM1", "NORM2", "Q", "Q_B", "K", "K_B", "V", "V_B", "G", "O",
-    "Q_NORM", "K_NORM", "SINK", "HEAD_NORM", "I", "I_B", "F", "F_B", "UP", "DOWN",
+    "Q_NORM", "K_NORM", "SINK", "HEAD_NORM", "I", "I_B", "F", "F_B", "UP", "DOWN", "NORM1B", "NORM2B",
+    "DQ", "DQ_NORM", "UQ", "DKV", "DKV_NORM", "UK", "UV", "GATE", "ROUTER", "EXPERT_GATE", "EXPERT_UP", "EXPERT_DOWN",
+    "SHARED_GATE", "SHARED_UP", "SHARED_DOWN",
 ]
 LAYERED_KIND = {name: i for i, name in enumerate(LAYERED_KINDS)}
-MIXERS = {"attention": 0, "mlstm": 1}
-MLPS = {None: 0, "relu2": 1}
+MIXERS = {"attention": 0, "mlstm": 1, "latent": 2}
+MLPS = {None: 0, "relu2": 1, "glu": 2, "moe": 3}
+GLUS = {"silu": 0, "clamped": 1}
 NORMS = {"rms": 0, "layer": 1}
+PLACES = {"post": 0, "sandwich": 1}
 MLSTM_AUTO, MLSTM_STEP = 0, 1
 
 EXPORTS = [
@@ -38,6 +42,7 @@ EXPORTS = [
     "arcb_engine_load_tensor", "arcb_session_workspace_bytes", "arcb_kv_cache_bytes",
     "arcb_session_create", "arcb_session_destroy", "arcb_prefill", "arcb_decode",
     "arcb_engine_create_layered", "arcb_session_feed", "arcb_session_step_logits", "arcb_session_finished",
+    "arcb_session_expand_rows",
     "arcb_session_poll", "arcb_engine_saturation_count", "arcb_session_attention_probe", "arcb_launch_count", "arcb_op_rmsnorm", "arcb_op_gemm",
     "arcb_op_gemm_residual", "arcb_gemm_splitk_scratch_bytes", "arcb_op_gemm_residual_splitk",
     "arcb_attn_scratch_bytes", "arcb_op_decode_attention", "arcb_op_decode_attention_static",
@@ -85,6 +90,7 @@ class PrefillArgs(C.Structure):
         ("n_segs", C.c_int32), ("d_seg_row0", C.c_void_p), ("d_seg_rows", C.c_void_p), ("d_seg_seq", C.c_void_p),
         ("d_seg_pos0", C.c_void_p), ("n_logit_rows", C.c_int32), ("d_logit_row", C.c_void_p),
         ("d_logits", C.c_void_p), ("d_residuals", C.c_void_p),
+        ("n_groups", C.c_int32), ("h_group_qblock", C.c_void_p), ("h_group_tile", C.c_void_p), ("d_tile_src", C.c_void_p),
     ]
 
 
@@ -93,13 +99,18 @@ class LayerDesc(C.Structure):
         ("mixer", C.c_int32), ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32),
         ("kv_from", C.c_int32), ("qkv_bias", C.c_int32), ("qk_norm", C.c_int32), ("sink", C.c_int32),
         ("out_gate", C.c_int32), ("scale", C.c_float), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_int32),
-        ("gate_cap", C.c_float), ("mlp", C.c_int32), ("d_ff", C.c_int32),
+        ("gate_cap", C.c_float), ("mlp", C.c_int32), ("d_ff", C.c_int32), ("window", C.c_int32),
+        ("q_rank", C.c_int32), ("kv_rank", C.c_int32), ("rot_dim", C.c_int32), ("rot_dims", C.c_int32),
+        ("rot_base", C.c_double), ("glu", C.c_int32), ("glu_limit", C.c_float), ("experts", C.c_int32), ("top", C.c_int32),
+        ("shared_ff", C.c_int32), ("shared_limit", C.c_float),
     ]
 
 
 class ModelDesc(C.Structure):
     _fields_ = [
-        ("width", C.c_int32), ("vocab", C.c_int32), ("n_layers", C.c_int32), ("norm", C.c_int32),
+        ("width", C.c_int32), ("vocab", C.c_int32), ("n_layers", C.c_int32),
+        ("norm_place", C.c_int32), ("loop_start", C.c_int32), ("loop_stop", C.c_int32), ("loop_times", C.c_int32),
+        ("norm", C.c_int32),
         ("act_format", C.c_int32), ("gemm_path", C.c_int32), ("attn_path", C.c_int32), ("mlstm_path", C.c_int32),
         ("fused_proj", C.c_int32), ("norm_eps", C.c_float), ("residual_alpha", C.c_float), ("logit_scale", C.c_float),
     ]
@@ -164,6 +175,7 @@ def load() -> C.CDLL:
     lib.arcb_session_feed.argtypes = [vp, i32, vp, vp, vp]
     lib.arcb_session_step_logits.argtypes = [vp, C.POINTER(vp), C.POINTER(i32)]
     lib.arcb_session_finished.argtypes = [vp, vp, vp]
+    lib.arcb_session_expand_rows.argtypes = [vp, C.POINTER(i32), C.POINTER(i32)]
     lib.arcb_prefill.argtypes = [vp, C.POINTER(PrefillArgs), vp]
     lib.arcb_decode.argtypes = [vp, i32, vp]
     lib.arcb_session_poll.argtypes = [vp, C.POINTER(i32), C.POINTER(i32), vp]

@@ -60,10 +60,13 @@ int arcb_launch_attn_gqa(AttnGqaArgs a, cudaStream_t stream) {
                 : a.fmt == 1 ? arcb_attn_gqa_dispatch_f16(a, grid, stream)
                              : arcb_attn_gqa_dispatch_bf16(a, grid, stream);
   arcb_count_launch(1);
-  if (e == cudaSuccess && a.n_splits > 1) {
-    const long long nb = ((long long)a.n_items * a.n_heads + 3) / 4;
-    e = arcb_launch(attn_gqa_combine_kernel, dim3((unsigned)nb), dim3(128), 0, stream, a);
-    arcb_count_launch(1);
-  }
+  if (e == cudaSuccess && a.n_splits > 1) return arcb_launch_attn_combine(a, stream);
+  return (int)e;
+}
+
+int arcb_launch_attn_combine(const AttnGqaArgs& a, cudaStream_t stream) {
+  const long long nb = ((long long)a.n_items * a.n_heads + 3) / 4;
+  const cudaError_t e = arcb_launch(attn_gqa_combine_kernel, dim3((unsigned)nb), dim3(128), 0, stream, a);
+  arcb_count_launch(1);
   return (int)e;
 }

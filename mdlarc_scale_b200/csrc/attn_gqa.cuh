@@ -12,7 +12,8 @@ struct AttnGqaArgs {
   long long gate_pitch;
   void* out;                  // [n_items][H][vdimp] activation format
   const int* item_seq;        // [n_items] cache row, null = item index
-  const int* item_len;        // [n_items] keys [0, len) are attended
+  const int* item_len;        // [n_items] keys [0, len) are attended,
+  int window;                 //   or the last `window` of them when window > 0
   const float* sink;          // optional [H]: exp(sink) joins the softmax denominator
   int n_items, n_heads, n_kv, dimp, vdimp, t_max, n_seqs, n_splits;
   float scale;
@@ -24,6 +25,8 @@ struct AttnGqaArgs {
 };
 
 int arcb_launch_attn_gqa(AttnGqaArgs a, cudaStream_t stream);
+// merges the splits in a.scratch ([item][head][split][vdimp + 4]: sums, reference maximum in log2 units, denominator)
+int arcb_launch_attn_combine(const AttnGqaArgs& a, cudaStream_t stream);
 // splits of a decode launch (upper bound used for the scratch when t_max is 0)
 int arcb_attn_gqa_splits(int n_items, int n_kv, int rep, int t_max);
 void arcb_count_launch(long long n);

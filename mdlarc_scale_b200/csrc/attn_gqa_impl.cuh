@@ -138,11 +138,11 @@ attn_gqa_kernel(AttnGqaArgs a) {
     len = 0;
   }
   if (len < 0) len = 0;
-  int begin = 0, end = len;
+  int begin = a.window > 0 ? max(0, len - a.window) : 0, end = len;
   if (a.n_splits > 1) {
-    int chunk = (len + a.n_splits - 1) / a.n_splits;
+    int chunk = (len - begin + a.n_splits - 1) / a.n_splits;
     chunk = (chunk + 15) & ~15;
-    begin = min(split * chunk, len);
+    begin = min(begin + split * chunk, len);
     end = min(begin + chunk, len);
   }
 

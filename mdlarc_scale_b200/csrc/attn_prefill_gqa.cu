@@ -5,7 +5,7 @@
 // Warps 0-3 are helpers (TMA producer, MMA issuer of A, MMA issuer of B, one idle); warps 4-11 serve tile A
 // and warps 12-19 tile B, two threads per query row: thread `half` owns keys [64 half, 64 half + 64) of every
 // 128-key tile and half of the output dims.  Per key tile j and Q tile x:
-//   TMA        K and V tiles as 128 x 64 boxes of the cache, 128-byte swizzle, ring shared by A and B
+//   TMA        K and V tiles as 128 x 64 boxes, 128-byte swizzle, rings shared by A and B
 //   MMA        S_x = Q_x K^T, fp32 in 128 TMEM columns
 //   softmax_x  scores to registers; reference maximum (raised only when exceeded by 2^8, O rescaled then);
 //              p = exp2(s c - m) in fp32, row sums in fp32; P rounded to the operand format and written over
@@ -15,6 +15,13 @@
 // it overwrites, and its completion implies that O(j) is complete.  While one Q tile is in the tensor core the
 // other tile's threads do exponentials.  A sink only joins the denominator at the end: rows are normalised by
 // l 2^m + 2^(sink log2 e).  The output gate multiplies the normalised row.  Every wait is bounded.
+//
+// A window hides keys from below: key tiles start at the first key the block's first row sees, and tile B skips
+// the tiles that lie ahead of its own first key.  With DR > 0 keys and values are those expanded from cached
+// latents: the first DP key columns and the values come from the expansion scratch, the last DR key columns,
+// which all heads share, from the latent cache itself.
+#include <type_traits>
+
 #include "attn_prefill_gqa.cuh"
 #include "flash_common.cuh"
 #include "gemm.cuh"
@@ -30,37 +37,63 @@ constexpr float LOG2E = 1.4426950408889634f;
 constexpr float RESCALE_THRESHOLD = 8.f;   // log2 units
 constexpr int BOX_BYTES = 128 * 64 * 2;    // one 128-row x 64-column box
 
-template <int DP, int VP>
+template <int DP, int DR, int VP>
 struct FgCfg {
-  static constexpr int Q_BYTES = (DP / 64) * BOX_BYTES;
-  static constexpr int K_BYTES = (DP / 64) * BOX_BYTES;
-  static constexpr int STAGE = K_BYTES + (VP / 64) * BOX_BYTES;
-  static constexpr int FIT = (208 * 1024 - 2 * Q_BYTES) / STAGE;
-  static constexpr int STAGES = FIT > 4 ? 4 : FIT;
-  static constexpr int SMEM = 2 * Q_BYTES + STAGES * STAGE + 1024 + 512;
+  static constexpr int QB = (DP + DR) / 64;  // boxes of a query (key) row
+  static constexpr int Q_BYTES = QB * BOX_BYTES;
+  static constexpr int K_BYTES = Q_BYTES;
+  static constexpr int V_BYTES = (VP / 64) * BOX_BYTES;
+  static constexpr int AVAIL = (DR > 0 ? 224 : 208) * 1024 - 2 * Q_BYTES;
+  static constexpr int FIT = AVAIL / (K_BYTES + V_BYTES);
+  static constexpr int V_STAGES = FIT > 4 ? 4 : FIT;
+  // one more key tile where it fits: the next tile's scores then do not wait for this tile's values
+  static constexpr int K_STAGES = V_STAGES < 4 && AVAIL >= (V_STAGES + 1) * K_BYTES + V_STAGES * V_BYTES ? V_STAGES + 1 : V_STAGES;
+  static_assert(V_STAGES >= 1, "a key tile and a value tile must fit");
+  static constexpr int TILES = 2 * Q_BYTES + K_STAGES * K_BYTES + V_STAGES * V_BYTES;
+  // DR = 0: 1 KB of alignment slack; exchange buffer and counts in static shared memory.  DR > 0 has no room for
+  // either: no static shared memory (the dynamic part then starts aligned, which is checked), maxima exchanged as
+  // bfloat16, denominators through the Q tile.
+  static constexpr int SMEM = DR > 0 ? TILES + 320 + 2 * 2 * 2 * BQ * 2 + 64 : TILES + 1024 + 512;
+  static_assert(SMEM + (DR > 0 ? 0 : 4096 + 64) <= 227 * 1024, "shared memory of one CTA");
   // S_A [0,128) S_B [128,256) O_A [256,256+VP) O_B; P_x of key half y occupies columns [64 y, 64 y + 32) of S_x
   static constexpr int TMEM_COLS = 512;
 };
 
-template <int DP, int VP, bool F16>
+template <int DP, int DR, int VP, bool F16>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_prefill_gqa_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
-                        const __grid_constant__ CUtensorMap tmap_v, AttnPrefillGqaArgs a, uint32_t idesc_qk,
-                        uint32_t idesc_pv) {
-  using C = FgCfg<DP, VP>;
+                        const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_r,
+                        AttnPrefillGqaArgs a, uint32_t idesc_qk, uint32_t idesc_pv) {
+  using C = FgCfg<DP, DR, VP>;
   pdl_launch_dependents();
   pdl_wait();   // the prologue below already reads the work list from global memory
-  extern __shared__ uint8_t smem_raw[];
-  __shared__ int s_max_cnt[16];
-  __shared__ float s_xchg[2][2][2][BQ];   // [tile parity][Q tile][half][row]
+  extern __shared__ __align__(1024) uint8_t smem_raw[];
+  using XT = typename std::conditional<(DR > 0), __nv_bfloat16, float>::type;
+  int* s_max_cnt;
+  XT (*s_xchg)[2][2][BQ];                 // [tile parity][Q tile][half][row]
+  if constexpr (DR == 0) {
+    __shared__ int static_cnt[16];
+    __shared__ XT static_xchg[2][2][2][BQ];
+    s_max_cnt = static_cnt;
+    s_xchg = static_xchg;
+  } else {
+    s_xchg = reinterpret_cast<XT (*)[2][2][BQ]>(smem_raw + C::TILES + 320);
+    s_max_cnt = reinterpret_cast<int*>(smem_raw + C::TILES + 320 + 2 * 2 * 2 * BQ * 2);
+    if (smem_u32(smem_raw) & 1023u) {
+      if (threadIdx.x == 0) arcb_set_error(a.err, ARCB_DEV_BAD_INDEX);
+      return;
+    }
+  }
   const uint32_t raw = smem_u32(smem_raw);
   const uint32_t base = (raw + 1023u) & ~1023u;
   uint8_t* base_ptr = smem_raw + (base - raw);
   const uint32_t q_smem = base;
-  const uint32_t kv_smem = base + 2 * C::Q_BYTES;
-  const uint32_t bar0 = kv_smem + C::STAGES * C::STAGE;
-  uint8_t* bar_ptr = base_ptr + 2 * C::Q_BYTES + C::STAGES * C::STAGE;
-  const uint32_t b_q = bar0, b_full = bar0 + 8, b_empty = b_full + 8 * C::STAGES, b_s = b_empty + 8 * C::STAGES,
+  const uint32_t k_smem = base + 2 * C::Q_BYTES;
+  const uint32_t v_smem = k_smem + C::K_STAGES * C::K_BYTES;
+  const uint32_t bar0 = v_smem + C::V_STAGES * C::V_BYTES;
+  uint8_t* bar_ptr = base_ptr + (bar0 - base);
+  const uint32_t b_q = bar0, b_kfull = bar0 + 8, b_kempty = b_kfull + 8 * C::K_STAGES, b_vfull = b_kempty + 8 * C::K_STAGES,
+                 b_vempty = b_vfull + 8 * C::V_STAGES, b_s = b_vempty + 8 * C::V_STAGES,
                  b_p = b_s + 16, b_o = b_p + 16, b_x = b_o + 16;     // b_x: 8 barriers, one per pair of warps of a row
   volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(bar_ptr + 256);
 
@@ -77,6 +110,9 @@ attn_prefill_gqa_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
   const int quarter = warp & 3;
   const int r = quarter * 32 + lane;
   int my_cnt = 0;
+  // first key tile, and the first one tile B reads (rows of a block are consecutive positions)
+  const int key0 = a.window > 0 && seq_ok ? max(0, a.kv_count[row0] - a.window) : 0;
+  const int j0_b = a.window > 0 && seq_ok && rows > BQ ? (max(0, a.kv_count[row0 + BQ] - a.window) - key0) / BKV : 0;
   if (warp >= 4) {
     const int qr = grp * BQ + r;
     if (qr < rows && seq_ok) my_cnt = a.kv_count[row0 + qr];
@@ -89,9 +125,13 @@ attn_prefill_gqa_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
   if (threadIdx.x == 0) {
     if (!seq_ok) arcb_set_error(a.err, ARCB_DEV_BAD_INDEX);
     mbar_init(b_q, 1);
-    for (int s = 0; s < C::STAGES; ++s) {
-      mbar_init(b_full + 8 * s, 1);
-      mbar_init(b_empty + 8 * s, 2);
+    for (int s = 0; s < C::K_STAGES; ++s) {
+      mbar_init(b_kfull + 8 * s, 1);
+      mbar_init(b_kempty + 8 * s, 2);
+    }
+    for (int s = 0; s < C::V_STAGES; ++s) {
+      mbar_init(b_vfull + 8 * s, 1);
+      mbar_init(b_vempty + 8 * s, 2);
     }
     for (int x = 0; x < 2; ++x) {
       mbar_init(b_s + 8 * x, 1);
@@ -103,6 +143,7 @@ attn_prefill_gqa_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
     tma_prefetch_desc(&tmap_q);
     tma_prefetch_desc(&tmap_k);
     tma_prefetch_desc(&tmap_v);
+    if (DR > 0) tma_prefetch_desc(&tmap_r);
   }
   if (warp == 1) {
     tmem_alloc(smem_u32(const_cast<uint32_t*>(tmem_slot)), C::TMEM_COLS);
@@ -118,7 +159,7 @@ attn_prefill_gqa_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
     cnt_a = max(cnt_a, s_max_cnt[i]);
     cnt_b = max(cnt_b, s_max_cnt[8 + i]);
   }
-  const int n_a = (cnt_a + BKV - 1) / BKV, n_b = (cnt_b + BKV - 1) / BKV;
+  const int n_a = (max(cnt_a - key0, 0) + BKV - 1) / BKV, n_b = (max(cnt_b - key0, 0) + BKV - 1) / BKV;
   const int n_tiles = max(n_a, n_b);
 
   if (warp < 4) {
@@ -126,30 +167,50 @@ attn_prefill_gqa_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
     if (warp == 0 && lane == 0 && n_tiles > 0) {
       // ---- TMA producer ----
       const bool two = rows > BQ;
-      const int kv0 = (seq * a.n_kv + h / (a.n_heads / a.n_kv)) * a.t_max;
+      int kv_row, k_col, v_col;
+      if (DR > 0) {
+        kv_row = a.kv0[blk] + key0;
+        k_col = h * DP;
+        v_col = a.v_col + h * VP;
+      } else {
+        kv_row = (seq * a.n_kv + h / (a.n_heads / a.n_kv)) * a.t_max + key0;
+        k_col = v_col = 0;
+      }
+      const int rot_row = seq * a.t_max + key0;
       mbar_expect_tx(b_q, two ? 2 * C::Q_BYTES : C::Q_BYTES);
 #pragma unroll
-      for (int c = 0; c < DP / 64; ++c) {
-        tma_load_2d(q_smem + c * BOX_BYTES, &tmap_q, a.q_col + h * DP + c * 64, row0, b_q);
-        if (two) tma_load_2d(q_smem + C::Q_BYTES + c * BOX_BYTES, &tmap_q, a.q_col + h * DP + c * 64, row0 + BQ, b_q);
+      for (int c = 0; c < C::QB; ++c) {
+        tma_load_2d(q_smem + c * BOX_BYTES, &tmap_q, a.q_col + h * (DP + DR) + c * 64, row0, b_q);
+        if (two) tma_load_2d(q_smem + C::Q_BYTES + c * BOX_BYTES, &tmap_q, a.q_col + h * (DP + DR) + c * 64, row0 + BQ, b_q);
       }
       for (int j = 0; j < n_tiles; ++j) {
-        const int s = j % C::STAGES;
-        if (!mbar_wait_bounded(b_empty + 8 * s, ((j / C::STAGES) & 1) ^ 1)) {
+        const int s = j % C::K_STAGES;
+        if (!mbar_wait_bounded(b_kempty + 8 * s, ((j / C::K_STAGES) & 1) ^ 1)) {
           arcb_set_error(a.err, ARCB_DEV_WAIT_TIMEOUT_MMA);
           break;
         }
-        const uint32_t dst = kv_smem + s * C::STAGE;
-        mbar_expect_tx(b_full + 8 * s, C::STAGE);
+        const uint32_t dst = k_smem + s * C::K_BYTES;
+        mbar_expect_tx(b_kfull + 8 * s, C::K_BYTES);
 #pragma unroll
-        for (int c = 0; c < DP / 64; ++c) tma_load_2d(dst + c * BOX_BYTES, &tmap_k, c * 64, kv0 + j * BKV, b_full + 8 * s);
+        for (int c = 0; c < DP / 64; ++c) tma_load_2d(dst + c * BOX_BYTES, &tmap_k, k_col + c * 64, kv_row + j * BKV, b_kfull + 8 * s);
 #pragma unroll
-        for (int c = 0; c < VP / 64; ++c) tma_load_2d(dst + C::K_BYTES + c * BOX_BYTES, &tmap_v, c * 64, kv0 + j * BKV, b_full + 8 * s);
+        for (int c = 0; c < DR / 64; ++c)
+          tma_load_2d(dst + (DP / 64 + c) * BOX_BYTES, &tmap_r, a.rot_col + c * 64, rot_row + j * BKV, b_kfull + 8 * s);
+        const int t = j % C::V_STAGES;
+        if (!mbar_wait_bounded(b_vempty + 8 * t, ((j / C::V_STAGES) & 1) ^ 1)) {
+          arcb_set_error(a.err, ARCB_DEV_WAIT_TIMEOUT_MMA);
+          break;
+        }
+        mbar_expect_tx(b_vfull + 8 * t, C::V_BYTES);
+#pragma unroll
+        for (int c = 0; c < VP / 64; ++c)
+          tma_load_2d(v_smem + t * C::V_BYTES + c * BOX_BYTES, &tmap_v, v_col + c * 64, kv_row + j * BKV, b_vfull + 8 * t);
       }
     } else if ((warp == 1 || warp == 2) && lane == 0 && n_tiles > 0) {
       // ---- MMA issuer of Q tile x ----
       const int x = warp - 1;
       const int n_x = x ? n_b : n_a;
+      const int j0 = x ? j0_b : 0;
       bool ok = true;
       auto wait_or_flag = [&](uint32_t bar, uint32_t parity, int code) {
         if (ok && !mbar_wait_bounded(bar, parity)) {
@@ -159,58 +220,72 @@ attn_prefill_gqa_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
       };
       const uint32_t t_s = tmem_base + x * 128, t_o = tmem_base + 256 + x * VP;
       auto mma_s = [&](int j) {
-        const uint32_t kst = kv_smem + (j % C::STAGES) * C::STAGE;
+        const uint32_t kst = k_smem + (j % C::K_STAGES) * C::K_BYTES;
 #pragma unroll
-        for (int c = 0; c < DP / 64; ++c) {
+        for (int c = 0; c < C::QB; ++c) {
           const uint64_t dq = umma_desc_k_sw128(q_smem + x * C::Q_BYTES + c * BOX_BYTES);
           const uint64_t dk = umma_desc_k_sw128(kst + c * BOX_BYTES);
 #pragma unroll
           for (int ks = 0; ks < 4; ++ks) umma_f16(t_s, dq + 2 * ks, dk + 2 * ks, idesc_qk, (c | ks) ? 1u : 0u);
         }
         umma_commit(b_s + 8 * x);
+        umma_commit(b_kempty + 8 * (j % C::K_STAGES));
       };
       auto mma_o = [&](int j) {
-        const uint32_t vst = kv_smem + (j % C::STAGES) * C::STAGE + C::K_BYTES;
+        const uint32_t vst = v_smem + (j % C::V_STAGES) * C::V_BYTES;
 #pragma unroll
         for (int c = 0; c < VP / 64; ++c) {
           const uint64_t dv = umma_desc_mn_sw128(vst + c * BOX_BYTES);
 #pragma unroll
           for (int ks = 0; ks < BKV / 16; ++ks)
-            umma_f16_ts(t_o + c * 64, t_s + (ks >> 2) * 64 + (ks & 3) * 8, dv + (uint64_t)(ks * (2048 >> 4)), idesc_pv, (j | ks) ? 1u : 0u);
+            umma_f16_ts(t_o + c * 64, t_s + (ks >> 2) * 64 + (ks & 3) * 8, dv + (uint64_t)(ks * (2048 >> 4)), idesc_pv, (j > j0 || ks) ? 1u : 0u);
         }
-        umma_commit(b_empty + 8 * (j % C::STAGES));
+        umma_commit(b_vempty + 8 * (j % C::V_STAGES));
       };
-      if (n_x > 0) {
+      auto wait_v = [&](int j) { wait_or_flag(b_vfull + 8 * (j % C::V_STAGES), (j / C::V_STAGES) & 1, ARCB_DEV_WAIT_TIMEOUT_TMA); };
+      auto wait_k = [&](int j) { wait_or_flag(b_kfull + 8 * (j % C::K_STAGES), (j / C::K_STAGES) & 1, ARCB_DEV_WAIT_TIMEOUT_TMA); };
+      // stages only the other tile uses: give them back in order as they land
+      auto pass = [&](int from, int to) {
+        for (int j = from; ok && j < to; ++j) {
+          wait_k(j);
+          if (ok) mbar_arrive(b_kempty + 8 * (j % C::K_STAGES));
+          wait_v(j);
+          if (ok) mbar_arrive(b_vempty + 8 * (j % C::V_STAGES));
+        }
+      };
+      if (n_x > j0) {
+        pass(0, j0);
         wait_or_flag(b_q, 0, ARCB_DEV_WAIT_TIMEOUT_TMA);
-        for (int j = 0; ok && j < n_x; ++j) {
-          if (j > 0) {
-            wait_or_flag(b_p + 8 * x, (j - 1) & 1, ARCB_DEV_WAIT_TIMEOUT_ACC);
+        for (int j = j0; ok && j < n_x; ++j) {
+          if (j > j0) {
+            wait_or_flag(b_p + 8 * x, (j - 1 - j0) & 1, ARCB_DEV_WAIT_TIMEOUT_ACC);
+            wait_v(j - 1);
             if (!ok) break;
             tc_fence_after();
             mma_o(j - 1);
           }
-          wait_or_flag(b_full + 8 * (j % C::STAGES), (j / C::STAGES) & 1, ARCB_DEV_WAIT_TIMEOUT_TMA);
+          wait_k(j);
           if (!ok) break;
           tc_fence_after();
           mma_s(j);
         }
-        wait_or_flag(b_p + 8 * x, (n_x - 1) & 1, ARCB_DEV_WAIT_TIMEOUT_ACC);
+        wait_or_flag(b_p + 8 * x, (n_x - 1 - j0) & 1, ARCB_DEV_WAIT_TIMEOUT_ACC);
+        wait_v(n_x - 1);
         if (ok) {
           tc_fence_after();
           mma_o(n_x - 1);
           umma_commit(b_o + 8 * x);
         }
-      }
-      // stages only the other tile uses: give them back in order as they land
-      for (int j = n_x; ok && j < n_tiles; ++j) {
-        wait_or_flag(b_full + 8 * (j % C::STAGES), (j / C::STAGES) & 1, ARCB_DEV_WAIT_TIMEOUT_TMA);
-        if (ok) mbar_arrive(b_empty + 8 * (j % C::STAGES));
+        pass(n_x, n_tiles);
+      } else {
+        pass(0, n_tiles);
       }
     }
   } else {
     reg_alloc_112();
     // ---- softmax / output threads: row r of Q tile grp, key half `half` ----
-    const int n_mine = grp ? n_b : n_a;
+    const int n_mine = grp ? n_b : n_a, j0 = grp ? j0_b : 0;
+    const int my_lo = a.window > 0 ? max(0, my_cnt - a.window) : 0;
     const uint32_t t_lane = tmem_base + ((uint32_t)(quarter * 32) << 16);
     const uint32_t t_s = t_lane + grp * 128 + half * 64;
     const uint32_t t_o = t_lane + 256 + grp * VP + half * (VP / 2);
@@ -219,26 +294,30 @@ attn_prefill_gqa_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
     float m_ref = -INFINITY, l = 0.f;
     bool ok = true;
     uint32_t xphase = 0;
-    auto exchange = [&](int slot, float mine, float& theirs) -> bool {
-      s_xchg[slot][grp][half][r] = mine;
+    // hands `mine` to the row's other thread; with bfloat16 both sides go on with the rounded values
+    auto exchange = [&](int slot, float& mine, float& theirs) -> bool {
+      const XT sent = (XT)mine;
+      mine = (float)sent;
+      s_xchg[slot][grp][half][r] = sent;
       tc_fence_before();
       mbar_arrive(xbar);
       const bool good = mbar_wait_bounded(xbar, xphase);
       tc_fence_after();
       xphase ^= 1u;
-      theirs = s_xchg[slot][grp][half ^ 1][r];
+      theirs = (float)s_xchg[slot][grp][half ^ 1][r];
       return good;
     };
-    for (int j = 0; j < n_mine; ++j) {
-      if (ok && !mbar_wait_bounded(b_s + 8 * grp, j & 1)) {
+    for (int j = j0; j < n_mine; ++j) {
+      if (ok && !mbar_wait_bounded(b_s + 8 * grp, (j - j0) & 1)) {
         arcb_set_error(a.err, ARCB_DEV_WAIT_TIMEOUT_ACC);
         ok = false;
       }
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       tc_fence_after();
-      const int n_valid = min(max(my_cnt - j * BKV, 0), BKV) - half * 64;
-      const bool full = __all_sync(0xffffffffu, n_valid >= 64);
+      const int tile_key = key0 + j * BKV + half * 64;            // visible: [v_lo, v_hi) of the thread's 64 keys
+      const int v_hi = my_cnt - tile_key, v_lo = my_lo - tile_key;
+      const bool full = __all_sync(0xffffffffu, v_hi >= 64 && v_lo <= 0);
       // 32 of the thread's 64 scores; hidden keys become -inf, whose exp2 is exactly 0
       auto load_scores = [&](int c, uint32_t (&sv)[32]) {
         tmem_ld_32x32(t_s + c * 32, sv);
@@ -246,7 +325,7 @@ attn_prefill_gqa_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
         if (!full) {
 #pragma unroll
           for (int i = 0; i < 32; ++i)
-            if (c * 32 + i >= n_valid) sv[i] = 0xff800000u;
+            if (c * 32 + i >= v_hi || c * 32 + i < v_lo) sv[i] = 0xff800000u;
         }
       };
       // the scores are read twice (maximum, then exponentials): tensor memory is quicker to read again than
@@ -261,7 +340,7 @@ attn_prefill_gqa_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
         for (int i = 2; i < 32; i += 2) mx2 = max3_f32(mx2, __uint_as_float(sv[i]), __uint_as_float(sv[i + 1]));
         raw_mx = fmaxf(raw_mx, mx2);
       }
-      const float mine = raw_mx == -INFINITY ? -INFINITY : raw_mx * sc;
+      float mine = raw_mx == -INFINITY ? -INFINITY : raw_mx * sc;
       float other;
       bool good = exchange(j & 1, mine, other);
       if (!good) arcb_set_error(a.err, ARCB_DEV_WAIT_TIMEOUT_ACC);
@@ -276,7 +355,7 @@ attn_prefill_gqa_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
       l *= alpha;
       const float m_safe = (m_ref == -INFINITY) ? 0.f : m_ref;
       const uint64_t sc2 = pack_f32x2(sc, sc), nm2 = pack_f32x2(-m_safe, -m_safe);
-      if (j > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {
+      if (j > j0 && __any_sync(0xffffffffu, alpha != 1.f)) {
         // S(j) was issued after P V(j - 1): O is complete and may be rescaled
 #pragma unroll
         for (int c = 0; c < VP / 64; ++c) {
@@ -315,9 +394,20 @@ attn_prefill_gqa_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
       mbar_arrive(b_p + 8 * grp);
     }
     float l_other = 0.f;
-    if (ok && n_mine > 0) {
-      bool good = exchange(n_mine & 1, l, l_other);
-      good = mbar_wait_bounded(b_o + 8 * grp, 0) && good;
+    if (ok && n_mine > j0) {
+      bool good;
+      if constexpr (DR == 0) {
+        good = exchange(n_mine & 1, l, l_other);
+        good = mbar_wait_bounded(b_o + 8 * grp, 0) && good;
+      } else {
+        // every product with this Q tile is complete: its shared memory is free
+        good = mbar_wait_bounded(b_o + 8 * grp, 0);
+        float* s_l = reinterpret_cast<float*>(base_ptr + grp * C::Q_BYTES);
+        s_l[half * BQ + r] = l;
+        mbar_arrive(xbar);
+        good = mbar_wait_bounded(xbar, xphase) && good;
+        l_other = s_l[(half ^ 1) * BQ + r];
+      }
       if (!good) arcb_set_error(a.err, ARCB_DEV_WAIT_TIMEOUT_ACC);
       ok = __all_sync(0xffffffffu, good);
     }
@@ -342,7 +432,7 @@ attn_prefill_gqa_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
       uint32_t oreg[32];
 #pragma unroll
       for (int i = 0; i < 32; ++i) oreg[i] = 0u;
-      if (ok && n_mine > 0) {
+      if (ok && n_mine > j0) {
         tc_fence_after();
         tmem_ld_32x32(t_o + c * 32, oreg);
         tmem_wait_ld_dep(oreg);
@@ -378,30 +468,37 @@ attn_prefill_gqa_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
   }
 }
 
-template <int DP, int VP>
+template <int DP, int DR, int VP>
 cudaError_t set_attr() {
-  cudaError_t e = cudaFuncSetAttribute(attn_prefill_gqa_kernel<DP, VP, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, FgCfg<DP, VP>::SMEM);
+  cudaError_t e = cudaFuncSetAttribute(attn_prefill_gqa_kernel<DP, DR, VP, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, FgCfg<DP, DR, VP>::SMEM);
   if (e != cudaSuccess) return e;
-  return cudaFuncSetAttribute(attn_prefill_gqa_kernel<DP, VP, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, FgCfg<DP, VP>::SMEM);
+  return cudaFuncSetAttribute(attn_prefill_gqa_kernel<DP, DR, VP, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, FgCfg<DP, DR, VP>::SMEM);
 }
 
-template <int DP, int VP>
+template <int DP, int DR, int VP>
 int launch(const AttnPrefillGqaArgs& a, cudaStream_t stream) {
+  using C = FgCfg<DP, DR, VP>;
   CUtensorMap tq, tk, tv;
   const uint64_t cache_rows = (uint64_t)a.n_seqs * a.n_kv * a.t_max;
+  const uint64_t kv_rows = DR > 0 ? (uint64_t)a.kv_rows : cache_rows;
   int r = arcb_make_tmap_2d_16b(&tq, a.q, (uint64_t)a.n_rows, (uint64_t)a.q_pitch, BQ, 64, a.act_f16);
   if (r) return 1000 + r;
-  r = arcb_make_tmap_2d_16b(&tk, a.k, cache_rows, DP, BKV, 64, a.act_f16);
+  r = arcb_make_tmap_2d_16b(&tk, a.k, kv_rows, DR > 0 ? (uint64_t)a.kv_pitch : DP, BKV, 64, a.act_f16);
   if (r) return 1000 + r;
-  r = arcb_make_tmap_2d_16b(&tv, a.v, cache_rows, VP, BKV, 64, a.act_f16);
+  r = arcb_make_tmap_2d_16b(&tv, a.v, kv_rows, DR > 0 ? (uint64_t)a.kv_pitch : VP, BKV, 64, a.act_f16);
   if (r) return 1000 + r;
+  CUtensorMap tr = tk;
+  if (DR > 0) {
+    r = arcb_make_tmap_2d_16b(&tr, a.k_rot, (uint64_t)a.n_seqs * a.t_max, (uint64_t)a.rot_pitch, BKV, 64, a.act_f16);
+    if (r) return 1000 + r;
+  }
   const int fmt = a.act_f16 ? 0 : 1;
   const uint32_t idesc_qk = umma_idesc_f16(BQ, BKV, fmt, fmt, 0, 0);
   const uint32_t idesc_pv = umma_idesc_f16(BQ, 64, fmt, fmt, 0, 1);   // V is MN-major, 64 columns a product
   const dim3 grid(a.n_heads, a.n_qblocks);
   const cudaError_t e =
-      a.act_f16 ? arcb_launch(attn_prefill_gqa_kernel<DP, VP, true>, grid, dim3(THREADS), FgCfg<DP, VP>::SMEM, stream, tq, tk, tv, a, idesc_qk, idesc_pv)
-                : arcb_launch(attn_prefill_gqa_kernel<DP, VP, false>, grid, dim3(THREADS), FgCfg<DP, VP>::SMEM, stream, tq, tk, tv, a, idesc_qk, idesc_pv);
+      a.act_f16 ? arcb_launch(attn_prefill_gqa_kernel<DP, DR, VP, true>, grid, dim3(THREADS), C::SMEM, stream, tq, tk, tv, tr, a, idesc_qk, idesc_pv)
+                : arcb_launch(attn_prefill_gqa_kernel<DP, DR, VP, false>, grid, dim3(THREADS), C::SMEM, stream, tq, tk, tv, tr, a, idesc_qk, idesc_pv);
   arcb_count_launch(1);
   return (int)e;
 }
@@ -413,23 +510,41 @@ bool arcb_attn_prefill_gqa_supported(int dimp, int vdimp, int n_seqs, int n_kv, 
   return scale > 0.f && dimp <= 128 && vdimp <= 128 && (long long)n_seqs * n_kv * t_max < (1ll << 31) - 256;
 }
 
+bool arcb_attn_prefill_latent_supported(int dimp, int rotp, int vdimp, int n_seqs, int t_max, float scale) {
+  return scale > 0.f && dimp <= 128 && rotp == 64 && vdimp <= 128 && (long long)n_seqs * t_max < (1ll << 31) - 256;
+}
+
 int arcb_attn_prefill_gqa_init() {
   cudaError_t e;
-  if ((e = set_attr<64, 64>()) != cudaSuccess) return (int)e;
-  if ((e = set_attr<64, 128>()) != cudaSuccess) return (int)e;
-  if ((e = set_attr<128, 64>()) != cudaSuccess) return (int)e;
-  if ((e = set_attr<128, 128>()) != cudaSuccess) return (int)e;
+  if ((e = set_attr<64, 0, 64>()) != cudaSuccess) return (int)e;
+  if ((e = set_attr<64, 0, 128>()) != cudaSuccess) return (int)e;
+  if ((e = set_attr<128, 0, 64>()) != cudaSuccess) return (int)e;
+  if ((e = set_attr<128, 0, 128>()) != cudaSuccess) return (int)e;
+  if ((e = set_attr<64, 64, 64>()) != cudaSuccess) return (int)e;
+  if ((e = set_attr<64, 64, 128>()) != cudaSuccess) return (int)e;
+  if ((e = set_attr<128, 64, 64>()) != cudaSuccess) return (int)e;
+  if ((e = set_attr<128, 64, 128>()) != cudaSuccess) return (int)e;
   return 0;
 }
 
 int arcb_launch_attn_prefill_gqa(const AttnPrefillGqaArgs& a, cudaStream_t stream) {
   if (a.n_qblocks <= 0) return 0;
   if (a.n_rows <= 0 || a.n_kv <= 0 || a.n_heads % a.n_kv || a.n_qblocks > 65535) return -1;
+  if (a.kv0) {
+    if (a.rotp != 64) return -1;
+    switch (a.dimp * 1000 + a.vdimp) {
+      case 64064: return launch<64, 64, 64>(a, stream);
+      case 64128: return launch<64, 64, 128>(a, stream);
+      case 128064: return launch<128, 64, 64>(a, stream);
+      case 128128: return launch<128, 64, 128>(a, stream);
+    }
+    return -1;
+  }
   switch (a.dimp * 1000 + a.vdimp) {
-    case 64064: return launch<64, 64>(a, stream);
-    case 64128: return launch<64, 128>(a, stream);
-    case 128064: return launch<128, 64>(a, stream);
-    case 128128: return launch<128, 128>(a, stream);
+    case 64064: return launch<64, 0, 64>(a, stream);
+    case 64128: return launch<64, 0, 128>(a, stream);
+    case 128064: return launch<128, 0, 64>(a, stream);
+    case 128128: return launch<128, 0, 128>(a, stream);
   }
   return -1;
 }

@@ -11,6 +11,38 @@ enum : int {
   EPI_SWIGLU = 3,     // h16[m][j] = silu(g+bg) * (u+bu)              (src/transformer.py:446-449)
   EPI_RELU2 = 4,      // out[m][n] = relu(acc)^2 in the activation format
   EPI_HEADS = 5,      // fused mixer projection of a layered model (ProjArgs)
+  EPI_ACT = 6,        // out[m][n] = acc in the activation format, optionally with rotated pairs (RotArgs)
+  EPI_GLU = 7,        // out[m][j] = glu(s g, s u) in the activation format, s a factor of the row (GluArgs)
+};
+
+// Rotation of neighbouring column pairs of every head: head h owns columns [h * head, (h + 1) * head), its
+// columns off + 2 i and off + 2 i + 1 (i < pairs) turn by the angle whose (cos, sin) is table[pos][i].
+struct RotArgs {
+  const float2* table;   // [t_max][pairs], null: nothing turns
+  const int* pos;        // [M], negative: position 0
+  int pairs, head, off, t_max;
+};
+
+// Gated linear unit of a packed gate/up product (64 gate columns, then the 64 matching up columns).
+struct GluArgs {
+  int kind;              // ARCB_GLU_*
+  float limit;           // ARCB_GLU_CLAMPED
+  const float* row;      // [M] factor of both products, null: 1; a factor 0 yields 0 whatever the products are
+};
+
+// Products whose rows or columns belong to groups.  All fields zero: one plain product.
+//   rows    : tile_src[t] is the A row of output rows [128 t, 128 t + 128) (null: 128 t); tile_group[t] picks the
+//             rows [group * group_rows, ...) of W; n_tiles (device) is the number of tiles that hold anything
+//   columns : columns [c n_group, (c + 1) n_group) read A columns [c a_group, c a_group + K)
+struct GroupArgs {
+  const int* tile_src;
+  const int* tile_group;
+  const int* n_tiles;
+  int group_rows;
+  long long w_rows;      // rows of W in all groups
+  int n_group, a_group;
+  int lda;               // row pitch of A in elements, 0: K
+  long long a_rows;      // rows of A, 0: M
 };
 
 // Fused projection of a mixer: the output columns are sections of whole heads, every head padded to
@@ -85,6 +117,10 @@ struct GemmEpilogue {
   int max_x, max_y, max_z;
   int* err;           // error word; word 1 counts 16-bit saturations
   ProjArgs pj;        // EPI_HEADS
+  int overwrite;      // EPI_RESID: x = acc instead of x += acc
+  RotArgs rot;        // EPI_ACT
+  GluArgs glu;        // EPI_GLU
+  GroupArgs grp;
 };
 
 struct RopeRow {
@@ -241,7 +277,7 @@ __device__ __forceinline__ void epi_qkv_chunk32(const GemmEpilogue& e, const Rop
 
 __device__ __forceinline__ void epi_resid_quad(const GemmEpilogue& e, int m, int n, float4 v) {
   float4* px = reinterpret_cast<float4*>(e.x + (size_t)m * e.N + n);
-  float4 r = *px;
+  float4 r = e.overwrite ? make_float4(0.f, 0.f, 0.f, 0.f) : *px;
   if (e.bias) {
     const float4 b = __ldg(reinterpret_cast<const float4*>(e.bias + n));
     v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
@@ -278,4 +314,67 @@ __device__ __forceinline__ void epi_swiglu_quad(const GemmEpilogue& e, int m, in
   pk.x = pack2_act_chk(silu_f(g.x) * u.x, silu_f(g.y) * u.y, e.act_f16, e.err);
   pk.y = pack2_act_chk(silu_f(g.z) * u.z, silu_f(g.w) * u.w, e.act_f16, e.err);
   *reinterpret_cast<uint2*>(reinterpret_cast<uint16_t*>(e.out16) + (size_t)m * (e.N >> 1) + j) = pk;
+}
+
+// ---- EPI_ACT ----
+// (cos, sin) row of the position of row m
+__device__ __forceinline__ const float2* rot_row(const GemmEpilogue& e, int m) {
+  const int p = min(max(e.rot.pos[m], 0), e.rot.t_max - 1);
+  return e.rot.table + (size_t)p * e.rot.pairs;
+}
+// columns n .. n + 3 (n % 4 == 0) of a row whose table row is cs
+__device__ __forceinline__ float4 rot_quad(const GemmEpilogue& e, const float2* cs, int n, float4 v) {
+  const int c = n % e.rot.head - e.rot.off;
+  if (c < 0) return v;
+  const int i = c >> 1;
+  float4 o = v;
+  if (i < e.rot.pairs) {
+    const float2 a = __ldg(cs + i);
+    o.x = v.x * a.x - v.y * a.y;
+    o.y = v.y * a.x + v.x * a.y;
+  }
+  if (i + 1 < e.rot.pairs) {
+    const float2 a = __ldg(cs + i + 1);
+    o.z = v.z * a.x - v.w * a.y;
+    o.w = v.w * a.x + v.z * a.y;
+  }
+  return o;
+}
+__device__ __forceinline__ void epi_act_quad(const GemmEpilogue& e, int m, int n, float4 v) {
+  if (e.rot.table) v = rot_quad(e, rot_row(e, m), n, v);
+  if (e.act_f16 == 1 && fmaxf(fmaxf(fabsf(v.x), fabsf(v.y)), fmaxf(fabsf(v.z), fabsf(v.w))) > 65504.f) arcb_count_saturation(e.err);
+  st_act4(e.out16, (size_t)m * e.N + n, v, e.act_f16);
+}
+
+// ---- EPI_GLU ----
+// EXACT: the accurate exponential and division (32-bit models), else the fast ones.
+template <bool EXACT>
+__device__ __forceinline__ float glu_sigmoid(float x) {
+  return EXACT ? 1.f / (1.f + expf(-x)) : __fdividef(1.f, 1.f + __expf(-x));
+}
+template <bool EXACT>
+__device__ __forceinline__ float glu_f(const GluArgs& a, float s, float g, float u) {
+  if (s == 0.f) return 0.f;
+  g *= s;
+  u *= s;
+  if (a.kind == 1) {
+    g = fminf(g, a.limit);
+    u = fminf(fmaxf(u, -a.limit), a.limit);
+    return g * glu_sigmoid<EXACT>(1.702f * g) * (u + 1.f);
+  }
+  return g * glu_sigmoid<EXACT>(g) * u;
+}
+__device__ __forceinline__ void epi_glu_quad(const GemmEpilogue& e, int m, int n, float4 g, float4 u) {
+  const float s = e.glu.row ? e.glu.row[m] : 1.f;
+  const size_t at = (size_t)m * (e.N >> 1) + (n >> 7) * 64 + (n & 127);
+  float4 v;
+  if (e.act_f16 == 2) {
+    v = make_float4(glu_f<true>(e.glu, s, g.x, u.x), glu_f<true>(e.glu, s, g.y, u.y), glu_f<true>(e.glu, s, g.z, u.z),
+                    glu_f<true>(e.glu, s, g.w, u.w));
+  } else {
+    v = make_float4(glu_f<false>(e.glu, s, g.x, u.x), glu_f<false>(e.glu, s, g.y, u.y), glu_f<false>(e.glu, s, g.z, u.z),
+                    glu_f<false>(e.glu, s, g.w, u.w));
+    if (e.act_f16 == 1 && fmaxf(fmaxf(fabsf(v.x), fabsf(v.y)), fmaxf(fabsf(v.z), fabsf(v.w))) > 65504.f) arcb_count_saturation(e.err);
+  }
+  st_act4(e.out16, at, v, e.act_f16);
 }

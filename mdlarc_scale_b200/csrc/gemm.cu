@@ -42,12 +42,13 @@ constexpr int EPI_STAGE_GROUP_BYTES = 128 * 32 * 4;
 template <int MODE>
 __host__ __device__ constexpr int epi_stage_bytes() {
   return (MODE == EPI_RESID || MODE == EPI_SWIGLU || MODE == EPI_QKV_ROPE || MODE == EPI_RELU2 ||
-          MODE == EPI_HEADS) ? 2 * EPI_STAGE_GROUP_BYTES : 0;
+          MODE == EPI_HEADS || MODE == EPI_ACT || MODE == EPI_GLU) ? 2 * EPI_STAGE_GROUP_BYTES : 0;
 }
 // epilogues that go through the staging buffers and the third tensor map
 template <int BN, int MODE>
 __host__ __device__ constexpr bool epi_staged() {
-  return MODE == EPI_RESID || MODE == EPI_RELU2 || MODE == EPI_HEADS || ((MODE == EPI_SWIGLU || MODE == EPI_QKV_ROPE) && BN == 256);
+  return MODE == EPI_RESID || MODE == EPI_RELU2 || MODE == EPI_HEADS || (MODE == EPI_ACT && BN >= 128) ||
+         ((MODE == EPI_SWIGLU || MODE == EPI_QKV_ROPE || MODE == EPI_GLU) && BN == 256);
 }
 
 // Residual epilogue: x[m][n] += acc[m][n] (+ bias[n]) for this CTA's 128 rows and this group's
@@ -89,7 +90,8 @@ __device__ __forceinline__ void epilogue_resid_tma(const GemmEpilogue& ep, const
     fence_proxy_async_smem();
     named_bar_sync(1 + col_half, 128);
     if (elected && m0 < ep.M) {
-      tma_reduce_add_2d(tmap_x, stage_smem, n0, m0);
+      if (ep.overwrite) tma_store_2d(tmap_x, stage_smem, n0, m0);
+      else tma_reduce_add_2d(tmap_x, stage_smem, n0, m0);
       bulk_commit_group();
     }
   }
@@ -99,10 +101,16 @@ __device__ __forceinline__ void epilogue_resid_tma(const GemmEpilogue& ep, const
 // columns) of a 256-column tile: h[m][j] = silu(g + bg) * (u + bu) for the group's 64 outputs.  The
 // group's four warps stage the 128 x 64 16-bit box (128-byte rows, XOR-swizzled 16-byte chunks) and
 // one thread issues a bulk tensor store, instead of 8-byte stores a row pitch apart.
+// MODE EPI_GLU: the linear unit of GluArgs with the row's factor instead (no biases).
+template <int MODE>
 __device__ __forceinline__ void epilogue_swiglu_tma(const GemmEpilogue& ep, const CUtensorMap* tmap_h, uint32_t t_grp,
                                                     int m0, int n_grp0, int grp, int row_in_tile,
                                                     uint32_t stage_smem, uint8_t* stage_ptr, bool elected) {
   if (n_grp0 >= ep.N) return;  // uniform over the group: tile tail beyond N
+  float row_factor = 1.f;
+  if constexpr (MODE == EPI_GLU) {
+    if (ep.glu.row && m0 + row_in_tile < ep.M) row_factor = __ldg(ep.glu.row + m0 + row_in_tile);
+  }
   uint8_t* my_row = stage_ptr + row_in_tile * 128;
   const int sw = row_in_tile & 7;
   if (elected) bulk_wait_read_all();   // the previous store has read the buffer
@@ -124,6 +132,11 @@ __device__ __forceinline__ void epilogue_swiglu_tma(const GemmEpilogue& ep, cons
                                __uint_as_float(rg[i + 3]));
         float4 u = make_float4(__uint_as_float(ru[i]), __uint_as_float(ru[i + 1]), __uint_as_float(ru[i + 2]),
                                __uint_as_float(ru[i + 3]));
+        if constexpr (MODE == EPI_GLU) {
+          w[2 * h] = pack2_act_chk(glu_f<false>(ep.glu, row_factor, g.x, u.x), glu_f<false>(ep.glu, row_factor, g.y, u.y), ep.act_f16, ep.err);
+          w[2 * h + 1] = pack2_act_chk(glu_f<false>(ep.glu, row_factor, g.z, u.z), glu_f<false>(ep.glu, row_factor, g.w, u.w), ep.act_f16, ep.err);
+          continue;
+        }
         if (ep.bias) {
           const float4 bg = __ldg(reinterpret_cast<const float4*>(ep.bias + n0 + i));
           const float4 bu = __ldg(reinterpret_cast<const float4*>(ep.bias + n0 + i + 64));
@@ -170,6 +183,57 @@ __device__ __forceinline__ void epilogue_relu2_tma(const GemmEpilogue& ep, const
         for (int i = 0; i < 4; ++i)
           w[i] = pack2_act_chk(relu2_f(__uint_as_float(r[8 * q + 2 * i])), relu2_f(__uint_as_float(r[8 * q + 2 * i + 1])),
                                ep.act_f16, ep.err);
+        *reinterpret_cast<uint4*>(my_row + (((half * 4 + q) ^ sw) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
+      }
+    }
+    fence_proxy_async_smem();
+    named_bar_sync(1 + grp, 128);
+    if (elected && m0 < ep.M) {
+      tma_store_2d(tmap_h, stage_smem, n0, m0);
+      bulk_commit_group();
+    }
+  }
+}
+
+// acc of this group's column half in the 16-bit activation format, pairs rotated where RotArgs says so (heads and
+// their rotated parts start at multiples of 64 columns, so a box is rotated as a whole or not at all).
+template <int BN>
+__device__ __forceinline__ void epilogue_act_tma(const GemmEpilogue& ep, const CUtensorMap* tmap_h, uint32_t t_row, int m0,
+                                                 bool row_ok, int n_tile0, int grp, int row_in_tile, uint32_t stage_smem,
+                                                 uint8_t* stage_ptr, bool elected) {
+  uint8_t* my_row = stage_ptr + row_in_tile * 128;
+  const int sw = row_in_tile & 7;
+  const float2* cs = (ep.rot.table && row_ok) ? rot_row(ep, m0 + row_in_tile) : nullptr;
+#pragma unroll 1
+  for (int b = grp * (BN / 128); b < (grp + 1) * (BN / 128); ++b) {
+    const int n0 = n_tile0 + b * 64;
+    if (n0 >= ep.N) break;               // uniform over the group
+    const int in_rot = cs ? n0 % ep.rot.head - ep.rot.off : -1;
+    if (elected) bulk_wait_read_all();   // the previous store has read the buffer
+    named_bar_sync(1 + grp, 128);
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      uint32_t r[32];
+      tmem_ld_32x32(t_row + b * 64 + half * 32, r);
+      tmem_wait_ld();
+      if (in_rot >= 0) {
+        const int i0 = (in_rot + half * 32) >> 1;
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          if (i0 + i < ep.rot.pairs) {
+            const float2 a = __ldg(cs + i0 + i);
+            const float x = __uint_as_float(r[2 * i]), y = __uint_as_float(r[2 * i + 1]);
+            r[2 * i] = __float_as_uint(x * a.x - y * a.y);
+            r[2 * i + 1] = __float_as_uint(y * a.x + x * a.y);
+          }
+        }
+      }
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        uint32_t w[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          w[i] = pack2_act_chk(__uint_as_float(r[8 * q + 2 * i]), __uint_as_float(r[8 * q + 2 * i + 1]), ep.act_f16, ep.err);
         *reinterpret_cast<uint4*>(my_row + (((half * 4 + q) ^ sw) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
       }
     }
@@ -426,7 +490,7 @@ __device__ __forceinline__ void epilogue_tile(const GemmEpilogue& ep, uint32_t t
   rr.kv_row = -1;
   rr.row16 = -1;
   if (MODE == EPI_QKV_ROPE && row_ok) rr = rope_row_ctx(ep, m);
-  if constexpr (MODE == EPI_SWIGLU) {
+  if constexpr (MODE == EPI_SWIGLU || MODE == EPI_GLU) {
     // gate columns [0,64) and up columns [64,128) of every 128-column group
     // BN = 256: each column half owns one 128-column group; BN = 128: one 32-column pair each
     const int g_begin = (BN == 256) ? col_half * 128 : 0, g_end = (BN == 256) ? g_begin + 128 : 128;
@@ -448,7 +512,8 @@ __device__ __forceinline__ void epilogue_tile(const GemmEpilogue& ep, uint32_t t
                                          __uint_as_float(rg[4 * q + 2]), __uint_as_float(rg[4 * q + 3]));
             const float4 u = make_float4(__uint_as_float(ru[4 * q]), __uint_as_float(ru[4 * q + 1]),
                                          __uint_as_float(ru[4 * q + 2]), __uint_as_float(ru[4 * q + 3]));
-            epi_swiglu_quad(ep, m, n0 + 4 * q, g, u);
+            if constexpr (MODE == EPI_GLU) epi_glu_quad(ep, m, n0 + 4 * q, g, u);
+            else epi_swiglu_quad(ep, m, n0 + 4 * q, g, u);
           }
         }
       }
@@ -472,6 +537,7 @@ __device__ __forceinline__ void epilogue_tile(const GemmEpilogue& ep, uint32_t t
             const int n = n0 + 4 * q;
             if constexpr (MODE == EPI_RESID) epi_resid_quad(ep, m, n, v);
             else if constexpr (MODE == EPI_RELU2) epi_relu2_quad(ep, m, n, v);
+            else if constexpr (MODE == EPI_ACT) epi_act_quad(ep, m, n, v);
             else epi_store_quad(ep, m, n, v);
           }
         }
@@ -532,6 +598,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
   pdl_wait();   // everything above touched only shared / tensor memory and the kernel's own parameters
+  const GroupArgs& g = ep.grp;
+  if (g.n_tiles) tiles_total = min(tiles_total, *g.n_tiles * tiles_n);
 
   if (warp == 0) {
     // ---- TMA producer ----
@@ -540,6 +608,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
       bool ok = true;
       for (int tile = blockIdx.x; ok && tile < tiles_total; tile += gridDim.x) {
         const int m_blk = tile / tiles_n, n_blk = tile - m_blk * tiles_n;
+        const int a_row = g.tile_src ? g.tile_src[m_blk] : m_blk * TC_BM;
+        const int w_row = n_blk * BN + (g.tile_group ? g.tile_group[m_blk] * g.group_rows : 0);
+        const int a_col = g.n_group ? n_blk * BN / g.n_group * g.a_group : 0;
         for (int kb = 0; kb < num_k; ++kb, ++kbt) {
           const int s = kbt % Cfg::STAGES;
           const uint32_t ph = (kbt / Cfg::STAGES) & 1;
@@ -553,8 +624,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
           const uint32_t full = bar_base + 8 * s;
           const uint32_t a_dst = base + s * Cfg::STAGE_BYTES;
           mbar_expect_tx(full, Cfg::STAGE_BYTES);
-          tma_load_2d(a_dst, &tmap_a, kb * TC_BK, m_blk * TC_BM, full);
-          tma_load_2d(a_dst + Cfg::A_BYTES, &tmap_b, kb * TC_BK, n_blk * BN, full);
+          tma_load_2d(a_dst, &tmap_a, a_col + kb * TC_BK, a_row, full);
+          tma_load_2d(a_dst + Cfg::A_BYTES, &tmap_b, kb * TC_BK, w_row, full);
         }
       }
     }
@@ -627,8 +698,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
         epilogue_relu2_tma<BN>(ep, &tmap_x, t_row, m_blk * TC_BM, n_blk * BN, col_half, row_in_tile,
                                base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
                                base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
-      else if constexpr (MODE == EPI_SWIGLU && BN == 256)
-        epilogue_swiglu_tma(ep, &tmap_x, t_row + col_half * 128, m_blk * TC_BM, n_blk * BN + col_half * 128, col_half,
+      else if constexpr (MODE == EPI_ACT && BN >= 128)
+        epilogue_act_tma<BN>(ep, &tmap_x, t_row, m_blk * TC_BM, row_ok, n_blk * BN, col_half, row_in_tile,
+                             base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
+                             base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
+      else if constexpr ((MODE == EPI_SWIGLU || MODE == EPI_GLU) && BN == 256)
+        epilogue_swiglu_tma<MODE>(ep, &tmap_x, t_row + col_half * 128, m_blk * TC_BM, n_blk * BN + col_half * 128, col_half,
                             row_in_tile, base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
                             base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
       else if constexpr (MODE == EPI_QKV_ROPE && BN == 256) {
@@ -739,6 +814,8 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constan
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
   pdl_wait();   // everything above touched only shared / tensor memory and the kernel's own parameters
+  const GroupArgs& g = ep.grp;       // a pair's two row tiles are of one group
+  if (g.n_tiles) tiles_total = min(tiles_total, (*g.n_tiles >> 1) * tiles_n);
 
   if (warp == 0) {
     // ---- TMA producer (both CTAs) ----
@@ -747,6 +824,9 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constan
       bool ok = true;
       for (int tile = pair; ok && tile < tiles_total; tile += n_pairs) {
         const int m_blk = tile / tiles_n, n_blk = tile - m_blk * tiles_n;
+        const int m_tile = 2 * m_blk + (int)rank;
+        const int a_row = g.tile_src ? g.tile_src[m_tile] : m_tile * 128;
+        const int w_row = n_blk * BN + (int)rank * 128 + (g.tile_group ? g.tile_group[m_tile] * g.group_rows : 0);
         for (int kb = 0; kb < num_k; ++kb, ++kbt) {
           const int s = kbt % Cfg::STAGES;
           const uint32_t ph = (kbt / Cfg::STAGES) & 1;
@@ -760,8 +840,8 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constan
           const uint32_t full = bar_base + 8 * s;
           const uint32_t a_dst = base + s * Cfg::STAGE_BYTES;
           if (rank == 0) mbar_expect_tx(full, 2 * Cfg::STAGE_BYTES);  // both CTAs' bytes land on CTA 0's barrier
-          tma_load_2d_2cta(a_dst, &tmap_a, kb * TC_BK, m_blk * 256 + (int)rank * 128, full);
-          tma_load_2d_2cta(a_dst + Cfg::A_BYTES, &tmap_b, kb * TC_BK, n_blk * BN + (int)rank * 128, full);
+          tma_load_2d_2cta(a_dst, &tmap_a, kb * TC_BK, a_row, full);
+          tma_load_2d_2cta(a_dst + Cfg::A_BYTES, &tmap_b, kb * TC_BK, w_row, full);
         }
       }
     }
@@ -830,8 +910,12 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constan
         epilogue_relu2_tma<BN>(ep, &tmap_x, t_row, m_blk * 256 + (int)rank * 128, n_blk * BN, col_half, row_in_tile,
                                base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
                                base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
-      else if constexpr (MODE == EPI_SWIGLU)
-        epilogue_swiglu_tma(ep, &tmap_x, t_row + col_half * 128, m_blk * 256 + (int)rank * 128,
+      else if constexpr (MODE == EPI_ACT)
+        epilogue_act_tma<BN>(ep, &tmap_x, t_row, m_blk * 256 + (int)rank * 128, row_ok, n_blk * BN, col_half, row_in_tile,
+                             base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
+                             base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
+      else if constexpr (MODE == EPI_SWIGLU || MODE == EPI_GLU)
+        epilogue_swiglu_tma<MODE>(ep, &tmap_x, t_row + col_half * 128, m_blk * 256 + (int)rank * 128,
                             n_blk * BN + col_half * 128, col_half, row_in_tile,
                             base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
                             base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
@@ -1049,7 +1133,8 @@ gemm_tc_splitk_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_c
         fence_proxy_async_smem();
         named_bar_sync(1 + col_half, 128);
         if (elected && m0 < ep.M) {
-          tma_reduce_add_2d(&tmap_x, stage_smem, n0, m0);
+          if (ep.overwrite) tma_store_2d(&tmap_x, stage_smem, n0, m0);
+          else tma_reduce_add_2d(&tmap_x, stage_smem, n0, m0);
           bulk_commit_group();
         }
       }
@@ -1081,6 +1166,12 @@ gemm_simt_kernel(const void* __restrict__ Av, const void* __restrict__ Wv, GemmE
   const int tid = threadIdx.x;
   const int tx = tid & 15, ty = tid >> 4;
   const int m0 = blockIdx.y * SM_BM, n0 = blockIdx.x * SM_BN;
+  const GroupArgs& g = ep.grp;
+  if (g.n_tiles && (m0 >> 7) >= *g.n_tiles) return;
+  const int a_row0 = g.tile_src ? g.tile_src[m0 >> 7] + (m0 & 127) : m0;
+  const long long a_rows = g.a_rows ? g.a_rows : ep.M;
+  const size_t lda = g.lda ? g.lda : K;
+  const size_t w_row0 = (size_t)n0 + (g.tile_group ? (size_t)g.tile_group[m0 >> 7] * g.group_rows : 0);
   float acc[2][8];
 #pragma unroll
   for (int i = 0; i < 2; ++i)
@@ -1092,14 +1183,14 @@ gemm_simt_kernel(const void* __restrict__ Av, const void* __restrict__ Wv, GemmE
   for (int k0 = 0; k0 < K; k0 += SM_BK) {
     {
       float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (m0 + a_row < ep.M) f = ld_act4(Av, (size_t)(m0 + a_row) * K + k0 + a_kq, a_fmt);
+      if (a_row0 + a_row < a_rows) f = ld_act4(Av, (size_t)(a_row0 + a_row) * lda + k0 + a_kq, a_fmt);
       As[a_kq + 0][a_row] = f.x;
       As[a_kq + 1][a_row] = f.y;
       As[a_kq + 2][a_row] = f.z;
       As[a_kq + 3][a_row] = f.w;
     }
     if (a_fmt == 2) {
-      const float4* src = reinterpret_cast<const float4*>(reinterpret_cast<const float*>(Wv) + (size_t)(n0 + w_n) * K + k0 + w_kh);
+      const float4* src = reinterpret_cast<const float4*>(reinterpret_cast<const float*>(Wv) + (w_row0 + w_n) * K + k0 + w_kh);
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const float4 f = __ldg(src + j);
@@ -1110,7 +1201,7 @@ gemm_simt_kernel(const void* __restrict__ Av, const void* __restrict__ Wv, GemmE
       }
     } else {
       const uint16_t* W = reinterpret_cast<const uint16_t*>(Wv);
-      const uint4* src = reinterpret_cast<const uint4*>(W + (size_t)(n0 + w_n) * K + k0 + w_kh);
+      const uint4* src = reinterpret_cast<const uint4*>(W + (w_row0 + w_n) * K + k0 + w_kh);
       const uint4 r0 = __ldg(src), r1 = __ldg(src + 1);
       const uint32_t w[8] = {r0.x, r0.y, r0.z, r0.w, r1.x, r1.y, r1.z, r1.w};
 #pragma unroll
@@ -1142,6 +1233,11 @@ gemm_simt_kernel(const void* __restrict__ Av, const void* __restrict__ Wv, GemmE
     const int n = n0 + 4 * tx;
     if constexpr (MODE == EPI_SWIGLU) {
       epi_swiglu_quad(ep, m, n, lo, hi);
+    } else if constexpr (MODE == EPI_GLU) {
+      epi_glu_quad(ep, m, n, lo, hi);
+    } else if constexpr (MODE == EPI_ACT) {
+      epi_act_quad(ep, m, n, lo);
+      epi_act_quad(ep, m, n + 64, hi);
     } else if constexpr (MODE == EPI_QKV_ROPE) {
       const RopeRow rr = rope_row_ctx(ep, m);
       epi_qkv_quad(ep, rr, m, n, lo);
@@ -1156,6 +1252,53 @@ gemm_simt_kernel(const void* __restrict__ Av, const void* __restrict__ Wv, GemmE
       epi_store_quad(ep, m, n, lo);
       epi_store_quad(ep, m, n + 64, hi);
     }
+  }
+}
+
+// CUDA-core kernel of products with column groups (EPI_ACT): 32 x 64 x 32 tiles, 256 threads, 2 rows x 4 columns
+// each; a tile lies inside one group.
+__global__ void __launch_bounds__(256)
+gemm_simt_groups_kernel(const void* __restrict__ Av, const void* __restrict__ Wv, GemmEpilogue ep, int K, int a_fmt) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float As[SM_BK][SM_BM + 1];
+  __shared__ __align__(16) float Ws[SM_BK][64 + 4];
+  const int tid = threadIdx.x;
+  const int tx = tid & 15, ty = tid >> 4;
+  const int m0 = blockIdx.y * SM_BM, n0 = blockIdx.x * 64;
+  const size_t a_col = (size_t)(n0 / ep.grp.n_group) * ep.grp.a_group;
+  float acc[2][4] = {};
+  const int a_row = tid >> 3, a_kq = (tid & 7) * 4;
+  const int w_n = tid >> 2, w_kq = (tid & 3) * 8;
+  for (int k0 = 0; k0 < K; k0 += SM_BK) {
+    float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (m0 + a_row < ep.M) f = ld_act4(Av, (size_t)(m0 + a_row) * ep.grp.lda + a_col + k0 + a_kq, a_fmt);
+    As[a_kq + 0][a_row] = f.x;
+    As[a_kq + 1][a_row] = f.y;
+    As[a_kq + 2][a_row] = f.z;
+    As[a_kq + 3][a_row] = f.w;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const float4 w = ld_act4(Wv, (size_t)(n0 + w_n) * K + k0 + w_kq + 4 * j, a_fmt);
+      Ws[w_kq + 4 * j + 0][w_n] = w.x;
+      Ws[w_kq + 4 * j + 1][w_n] = w.y;
+      Ws[w_kq + 4 * j + 2][w_n] = w.z;
+      Ws[w_kq + 4 * j + 3][w_n] = w.w;
+    }
+    __syncthreads();
+#pragma unroll 8
+    for (int k = 0; k < SM_BK; ++k) {
+      const float a0 = As[k][2 * ty], a1 = As[k][2 * ty + 1];
+      const float4 w = *reinterpret_cast<const float4*>(&Ws[k][4 * tx]);
+      acc[0][0] += a0 * w.x; acc[0][1] += a0 * w.y; acc[0][2] += a0 * w.z; acc[0][3] += a0 * w.w;
+      acc[1][0] += a1 * w.x; acc[1][1] += a1 * w.y; acc[1][2] += a1 * w.z; acc[1][3] += a1 * w.w;
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int m = m0 + 2 * ty + i;
+    if (m < ep.M) epi_act_quad(ep, m, n0 + 4 * tx, make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]));
   }
 }
 
@@ -1253,6 +1396,12 @@ int arcb_gemm_init() {
   if ((e = set_tc_smem_attr<EPI_SWIGLU>()) != cudaSuccess) return (int)e;
   if ((e = set_tc_smem_attr<EPI_RELU2>()) != cudaSuccess) return (int)e;
   if ((e = set_tc_smem_attr<EPI_HEADS>()) != cudaSuccess) return (int)e;
+  if ((e = set_tc_smem_attr<EPI_ACT>()) != cudaSuccess) return (int)e;
+  if ((e = cudaFuncSetAttribute(gemm_tc_kernel<64, EPI_ACT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                TcCfg<64>::SMEM_BYTES + epi_stage_bytes<EPI_ACT>())) != cudaSuccess) return (int)e;
+  if ((e = set_tc_smem_attr<EPI_GLU>()) != cudaSuccess) return (int)e;
+  if ((e = set_tc2_smem_attr<EPI_ACT>()) != cudaSuccess) return (int)e;
+  if ((e = set_tc2_smem_attr<EPI_GLU>()) != cudaSuccess) return (int)e;
   if ((e = set_tc2_smem_attr<EPI_HEADS>()) != cudaSuccess) return (int)e;
   if ((e = set_tc2_smem_attr<EPI_STORE_F32>()) != cudaSuccess) return (int)e;
   if ((e = set_tc2_smem_attr<EPI_RELU2>()) != cudaSuccess) return (int)e;
@@ -1347,7 +1496,24 @@ template <int MODE>
 static int launch_gemm_mode(const void* a16, const void* w16, const GemmEpilogue& ep, int K,
                             int act_f16, bool use_tc, int tc_variant, cudaStream_t stream) {
   const int M = ep.M, N = ep.N;
+  const GroupArgs& g = ep.grp;
+  const uint64_t a_rows = g.a_rows ? (uint64_t)g.a_rows : (uint64_t)M, a_cols = g.lda ? (uint64_t)g.lda : (uint64_t)K;
+  const uint64_t w_rows = g.w_rows ? (uint64_t)g.w_rows : (uint64_t)N;
   if (use_tc) {
+    if constexpr (MODE == EPI_ACT) {
+      if (g.n_group) {   // a tile lies inside one column group
+        const int bn = g.n_group % 128 == 0 ? 128 : 64;
+        CUtensorMap ta, tb, tx;
+        int r = arcb_make_tmap_2d_16b(&ta, a16, a_rows, a_cols, TC_BM, TC_BK, act_f16);
+        if (!r) r = arcb_make_tmap_2d_16b(&tb, w16, w_rows, (uint64_t)K, bn, TC_BK, act_f16);
+        if (!r) r = arcb_make_tmap_2d_16b(&tx, ep.out16, (uint64_t)M, (uint64_t)N, 128, 64, act_f16);
+        if (r) return 1000 + r;
+        const cudaError_t le = bn == 128 ? launch_tc<128, MODE>(ta, tb, tx, ta, ta, ep, K, act_f16, stream)
+                                         : launch_tc<64, MODE>(ta, tb, tx, ta, ta, ep, K, act_f16, stream);
+        arcb_count_launch(1);
+        return (int)le;
+      }
+    }
     // 128 x 256 tiles (one CTA per SM, persistent) unless that leaves most SMs without a tile
     const int sms = num_sms();
     const int tiles256 = ((N + 255) / 256) * ((M + TC_BM - 1) / TC_BM);
@@ -1359,7 +1525,7 @@ static int launch_gemm_mode(const void* a16, const void* w16, const GemmEpilogue
     const int mp = max_pairs();
     const bool pair = allow256 && mp > 0 && (tc_variant == 2 || (tc_variant == 0 && tiles2 * 10 >= mp * 7));
     CUtensorMap ta, tb;
-    int r = arcb_make_tmap_2d_16b(&ta, a16, (uint64_t)M, (uint64_t)K, TC_BM, TC_BK, act_f16);
+    int r = arcb_make_tmap_2d_16b(&ta, a16, a_rows, a_cols, TC_BM, TC_BK, act_f16);
     if (r) return 1000 + r;
     if (MODE == EPI_RESID && ep.splitk_scratch && tc_variant == 0) {
       const int bn = arcb_gemm_splitk_bn(M, N, K);
@@ -1375,7 +1541,7 @@ static int launch_gemm_mode(const void* a16, const void* w16, const GemmEpilogue
         return (int)le;
       }
     }
-    r = arcb_make_tmap_2d_16b(&tb, w16, (uint64_t)N, (uint64_t)K, (wide && !pair) ? 256 : 128, TC_BK, act_f16);
+    r = arcb_make_tmap_2d_16b(&tb, w16, w_rows, (uint64_t)K, (wide && !pair) ? 256 : 128, TC_BK, act_f16);
     if (r) return 1000 + r;
     CUtensorMap tx = ta;  // only the residual epilogue reads it
     if (MODE == EPI_RESID) {
@@ -1384,10 +1550,10 @@ static int launch_gemm_mode(const void* a16, const void* w16, const GemmEpilogue
     } else if (MODE == EPI_HEADS) {
       r = arcb_make_tmap_2d_16b(&tx, ep.pj.out, (uint64_t)M, (uint64_t)N, 128, 64, act_f16);
       if (r) return 1000 + r;
-    } else if (MODE == EPI_RELU2) {
+    } else if (MODE == EPI_RELU2 || MODE == EPI_ACT) {
       r = arcb_make_tmap_2d_16b(&tx, ep.out16, (uint64_t)M, (uint64_t)N, 128, 64, act_f16);
       if (r) return 1000 + r;
-    } else if (MODE == EPI_SWIGLU && (pair || wide)) {
+    } else if ((MODE == EPI_SWIGLU || MODE == EPI_GLU) && (pair || wide)) {
       // h16 [M][N / 2], 128 x 64 boxes (one accumulator group's outputs)
       r = arcb_make_tmap_2d_16b(&tx, ep.out16, (uint64_t)M, (uint64_t)(N / 2), 128, 64, act_f16);
       if (r) return 1000 + r;
@@ -1426,6 +1592,12 @@ static int launch_gemm_mode(const void* a16, const void* w16, const GemmEpilogue
     arcb_count_launch(1);
     return (int)le;
   }
+  if (MODE == EPI_ACT && g.n_group) {
+    const cudaError_t le = arcb_launch(gemm_simt_groups_kernel, dim3(N / 64, (M + SM_BM - 1) / SM_BM), dim3(256), 0, stream, a16,
+                                       w16, ep, K, act_f16);
+    arcb_count_launch(1);
+    return (int)le;
+  }
   dim3 grid(N / SM_BN, (M + SM_BM - 1) / SM_BM);
   const cudaError_t le = arcb_launch(gemm_simt_kernel<MODE>, grid, dim3(256), 0, stream,
                                      a16, w16, ep, K, act_f16);
@@ -1447,6 +1619,10 @@ int arcb_launch_gemm(const void* a16, const void* w16, const GemmEpilogue& ep, i
     case EPI_HEADS:   // needs whole rows of a head in one thread: tensor-core kernels only
       if (!use_tc) return -1;
       return launch_gemm_mode<EPI_HEADS>(a16, w16, ep, K, act_f16, use_tc, tc_variant, stream);
+    case EPI_ACT:
+      if (ep.grp.n_group && (ep.grp.n_group % 64 || !ep.grp.lda || ep.grp.tile_src || ep.grp.tile_group)) return -1;
+      return launch_gemm_mode<EPI_ACT>(a16, w16, ep, K, act_f16, use_tc, tc_variant, stream);
+    case EPI_GLU: return launch_gemm_mode<EPI_GLU>(a16, w16, ep, K, act_f16, use_tc, tc_variant, stream);
     case EPI_RELU2: return launch_gemm_mode<EPI_RELU2>(a16, w16, ep, K, act_f16, use_tc, tc_variant, stream);
   }
   return -1;

@@ -1,6 +1,8 @@
 // Row-wise kernels of layered models:
 //   lm_embed / step_begin : embedding -> residual stream (+ the decode step's positions)
 //   lm_norm               : norm of the residual stream -> GEMM operand, and the scaled residual in place
+//   sandwich_norm         : norm of a sublayer's output, residual sum and the next sublayer's norm in one pass
+//   latent_prep           : query latent, cached latent and rotated key part from their fp32 projections
 //   proj_prep             : head norms, query gain, gates and cache writes of a projection left in fp32
 //   pick                  : logit scale, argmax or temperature / top-k sampling, decode bookkeeping
 // Norms, gates, angles and the residual are fp32 throughout; fmt selects the operand format.
@@ -148,6 +150,170 @@ lm_norm_kernel(LmNormArgs a) {
   else if (a.pitch <= 128 * 10) norm_row_regs<10>(a, x, row, lane);
   else if (a.pitch <= 128 * 16) norm_row_regs<16>(a, x, row, lane);
   else norm_row_loop(a, x, row, lane);
+}
+
+// Sum over a CTA of WARPS warps; every thread gets it.  Two calls in a row need different `sm`.
+template <int WARPS>
+__device__ __forceinline__ float cta_sum(float v, float* sm) {
+  v = warp_sum(v);
+  if constexpr (WARPS == 1) return v;
+  if ((threadIdx.x & 31) == 0) sm[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = sm[0];
+#pragma unroll
+  for (int i = 1; i < WARPS; ++i) t += sm[i];
+  return t;
+}
+
+__device__ __forceinline__ float sum_sq(float4 v) { return (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w); }
+
+// One CTA of four warps per row; NV float4 per thread hold the row (REGS) or every pass reads it again.
+template <int NV, bool REGS>
+__global__ void __launch_bounds__(128)
+sandwich_norm_kernel(SandwichArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float sm[2][4];
+  const int row = blockIdx.x, tid = threadIdx.x;
+  float* x = a.x + (size_t)row * a.pitch;
+  const float* y = a.y ? a.y + (size_t)row * a.pitch : nullptr;
+  const float inv_n = 1.f / (float)a.width;
+  auto sublayer = [&](int i) {
+    float4 v = y ? *reinterpret_cast<const float4*>(y + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    if (a.ye)
+      for (int k = 0; k < a.top; ++k) {
+        const float4 e = ld_act4(a.ye, (size_t)a.slot[(size_t)row * a.top + k] * a.pitch + i, a.fmt);
+        v.x += e.x; v.y += e.y; v.z += e.z; v.w += e.w;
+      }
+    return v;
+  };
+  auto added = [&](int i, float4 v, float inv) {
+    const float4 g = __ldg(reinterpret_cast<const float4*>(a.w_out + i));
+    const float4 r = *reinterpret_cast<const float4*>(x + i);
+    return make_float4(r.x + (v.x * inv) * g.x, r.y + (v.y * inv) * g.y, r.z + (v.z * inv) * g.z, r.w + (v.w * inv) * g.w);
+  };
+  auto dense = [&](int i, float4 v) {
+    float* d = a.dense + (size_t)row * a.width;
+    if (i < a.width) d[i] = v.x;
+    if (i + 1 < a.width) d[i + 1] = v.y;
+    if (i + 2 < a.width) d[i + 2] = v.z;
+    if (i + 3 < a.width) d[i + 3] = v.w;
+  };
+  const float* emb = a.embed ? a.embed + (size_t)min(max(a.tokens[row], 0), a.vocab - 1) * a.pitch : nullptr;
+  auto with_embed = [&](int i, float4 v) {
+    if (emb) {
+      const float4 e = __ldg(reinterpret_cast<const float4*>(emb + i));
+      v.x += e.x; v.y += e.y; v.z += e.z; v.w += e.w;
+    }
+    return v;
+  };
+  auto write_xn = [&](int i, float4 v, float inv) {
+    const float4 g = __ldg(reinterpret_cast<const float4*>(a.w_in + i));
+    st_act4(a.xn, (size_t)row * a.pitch + i, make_float4((v.x * inv) * g.x, (v.y * inv) * g.y, (v.z * inv) * g.z, (v.w * inv) * g.w), a.fmt);
+  };
+  // padding columns are zero in y, x, the embedding and the gains
+  if constexpr (REGS) {
+    float4 v[NV];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int i = (tid + k * 128) * 4;
+      v[k] = i < a.pitch ? sublayer(i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss += sum_sq(v[k]);
+    }
+    float inv = 1.f / sqrtf(cta_sum<4>(ss, sm[0]) * inv_n + a.eps);
+    ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int i = (tid + k * 128) * 4;
+      if (i >= a.pitch) continue;
+      v[k] = added(i, v[k], inv);
+      if (a.dense) dense(i, v[k]);
+      v[k] = with_embed(i, v[k]);
+      *reinterpret_cast<float4*>(x + i) = v[k];
+      ss += sum_sq(v[k]);
+    }
+    if (!a.w_in) return;
+    inv = 1.f / sqrtf(cta_sum<4>(ss, sm[1]) * inv_n + a.eps);
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int i = (tid + k * 128) * 4;
+      if (i < a.pitch) write_xn(i, v[k], inv);
+    }
+  } else {
+    float ss = 0.f;
+    for (int i = tid * 4; i < a.pitch; i += 512) ss += sum_sq(sublayer(i));
+    float inv = 1.f / sqrtf(cta_sum<4>(ss, sm[0]) * inv_n + a.eps);
+    ss = 0.f;
+    for (int i = tid * 4; i < a.pitch; i += 512) {
+      float4 v = added(i, sublayer(i), inv);
+      if (a.dense) dense(i, v);
+      v = with_embed(i, v);
+      *reinterpret_cast<float4*>(x + i) = v;
+      ss += sum_sq(v);
+    }
+    if (!a.w_in) return;
+    inv = 1.f / sqrtf(cta_sum<4>(ss, sm[1]) * inv_n + a.eps);
+    for (int i = tid * 4; i < a.pitch; i += 512) write_xn(i, *reinterpret_cast<const float4*>(x + i), inv);
+  }
+}
+
+// One CTA per row, WARPS warps; both norms' sums in one pass, then the row is read again (L1).
+template <int WARPS>
+__global__ void __launch_bounds__(WARPS * 32)
+latent_prep_kernel(LatentPrepArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float sm[2][WARPS];
+  constexpr int STEP = WARPS * 32 * 4;
+  const int row = blockIdx.x, tid = threadIdx.x;
+  const float* p = a.proj + (size_t)row * a.pitch;
+  float sq = 0.f, sc = 0.f;
+  for (int i = tid * 4; i < a.q_rankp; i += STEP) sq += sum_sq(*reinterpret_cast<const float4*>(p + i));
+  for (int i = tid * 4; i < a.kv_rankp; i += STEP) sc += sum_sq(*reinterpret_cast<const float4*>(p + a.off_c + i));
+  const float iq = 1.f / sqrtf(cta_sum<WARPS>(sq, sm[0]) / (float)a.q_rank + a.eps);
+  const float ic = 1.f / sqrtf(cta_sum<WARPS>(sc, sm[1]) / (float)a.kv_rank + a.eps);
+  auto normed = [&](const float* src, const float* w, int i, float inv) {
+    const float4 v = *reinterpret_cast<const float4*>(src + i), g = __ldg(reinterpret_cast<const float4*>(w + i));
+    return make_float4((v.x * inv) * g.x, (v.y * inv) * g.y, (v.z * inv) * g.z, (v.w * inv) * g.w);
+  };
+  for (int i = tid * 4; i < a.q_rankp; i += STEP)
+    st_act4(a.cq, (size_t)row * a.q_rankp + i, normed(p, a.q_norm, i, iq), a.fmt);
+  const int pos = a.pos[row], seq = a.seq ? a.seq[row] : row;
+  if (pos < 0) return;
+  if (pos >= a.t_max || seq < 0 || seq >= a.n_seqs) {
+    if (tid == 0) arcb_set_error(a.err, ARCB_DEV_BAD_INDEX);
+    return;
+  }
+  const size_t at = ((size_t)seq * a.t_max + pos) * (a.kv_rankp + a.rotp);
+  for (int i = tid * 4; i < a.kv_rankp; i += STEP) st_act4(a.cache, at + i, normed(p + a.off_c, a.kv_norm, i, ic), a.fmt);
+  for (int i = tid * 4; i < a.rotp; i += STEP) {
+    const float4 v = *reinterpret_cast<const float4*>(p + a.off_r + i);
+    float4 o = v;
+    const int q = i >> 1;
+    if (q < a.pairs) {
+      const float2 c = __ldg(a.rot + (size_t)pos * a.pairs + q);
+      o.x = v.x * c.x - v.y * c.y;
+      o.y = v.y * c.x + v.x * c.y;
+    }
+    if (q + 1 < a.pairs) {
+      const float2 c = __ldg(a.rot + (size_t)pos * a.pairs + q + 1);
+      o.z = v.z * c.x - v.w * c.y;
+      o.w = v.w * c.x + v.z * c.y;
+    }
+    st_act4(a.cache, at + a.kv_rankp + i, o, a.fmt);
+  }
+}
+
+// Angles in double precision: a position times a frequency loses nothing before the sine.
+__global__ void rot_table_kernel(float2* table, int t_max, int pairs, int dims, double base) {
+  const long long n = (long long)t_max * pairs;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+    const int p = (int)(i / pairs), k = (int)(i - (long long)p * pairs);
+    double s, c;
+    sincos(p * pow(base, -2.0 * k / dims), &s, &c);
+    table[i] = make_float2((float)c, (float)s);
+  }
 }
 
 // One warp per (row, head of a section): 4 consecutive columns per lane and 128-column step.
@@ -438,7 +604,59 @@ __global__ void pack_blocks_kernel(const float* __restrict__ src, void* __restri
   }
 }
 
+__global__ void pack_heads_t_kernel(const float* __restrict__ src, void* __restrict__ dst, int heads, int rb, int rbp, int cols,
+                                    long long dst_pitch, int container) {
+  const long long n = (long long)heads * rb * cols;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / cols;
+    const int c = (int)(i - r * cols), h = (int)(r / rb), d = (int)(r - (long long)h * rb);
+    const long long at = ((long long)h * rbp + c) * dst_pitch + d;
+    if (container == 2) reinterpret_cast<float*>(dst)[at] = src[i];
+    else st_act(dst, at, __bfloat162float(__float2bfloat16_rn(src[i])), container);
+  }
+}
+
 }  // namespace
+
+int arcb_launch_sandwich_norm(const SandwichArgs& a, cudaStream_t stream) {
+  if (a.rows <= 0) return 0;
+  if (a.pitch % 128) return -1;
+  const dim3 grid(a.rows), block(128);
+  const cudaError_t e = a.pitch <= 512 * 2   ? arcb_launch(sandwich_norm_kernel<2, true>, grid, block, 0, stream, a)
+                        : a.pitch <= 512 * 4 ? arcb_launch(sandwich_norm_kernel<4, true>, grid, block, 0, stream, a)
+                        : a.pitch <= 512 * 8 ? arcb_launch(sandwich_norm_kernel<8, true>, grid, block, 0, stream, a)
+                                             : arcb_launch(sandwich_norm_kernel<1, false>, grid, block, 0, stream, a);
+  arcb_count_launch(1);
+  return (int)e;
+}
+
+int arcb_launch_latent_prep(const LatentPrepArgs& a, cudaStream_t stream) {
+  if (a.rows <= 0) return 0;
+  if (a.q_rankp % 4 || a.kv_rankp % 4 || a.rotp % 4 || a.off_c % 4 || a.off_r % 4 || a.pitch % 4) return -1;
+  const cudaError_t e = arcb_launch(latent_prep_kernel<4>, dim3(a.rows), dim3(128), 0, stream, a);
+  arcb_count_launch(1);
+  return (int)e;
+}
+
+int arcb_launch_rot_table(float2* table, int t_max, int dims, double base, cudaStream_t stream) {
+  if (t_max <= 0 || dims < 2) return 0;
+  long long blocks = ((long long)t_max * (dims / 2) + 255) / 256;
+  if (blocks > 148 * 8) blocks = 148 * 8;
+  rot_table_kernel<<<(unsigned)blocks, 256, 0, stream>>>(table, t_max, dims / 2, dims, base);
+  arcb_count_launch(1);
+  return (int)cudaGetLastError();
+}
+
+int arcb_launch_pack_heads_t(const float* src, void* dst, int heads, int rb, int rbp, int cols, long long dst_pitch, int container,
+                             cudaStream_t stream) {
+  const long long n = (long long)heads * rb * cols;
+  if (n <= 0) return 0;
+  long long blocks = (n + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  pack_heads_t_kernel<<<(unsigned)blocks, 256, 0, stream>>>(src, dst, heads, rb, rbp, cols, dst_pitch, container);
+  arcb_count_launch(1);
+  return (int)cudaGetLastError();
+}
 
 int arcb_launch_lm_embed(const LmEmbedArgs& a, cudaStream_t stream) {
   if (a.rows <= 0) return 0;

@@ -46,6 +46,42 @@ struct LmNormArgs {
   float* dense;            // optional [rows][width]: y, without padding
 };
 
+// Sandwich norms, one sublayer to the next: x += norm(y) * w_out, then xn = norm(x) * w_in in the activation format.
+// y is the sum of a fp32 row and of `top` rows of an expert product.
+struct SandwichArgs {
+  int rows, width, pitch, fmt, top;
+  float eps;
+  float* x;                // [rows][pitch]
+  const float* y;          // [rows][pitch], null: zero
+  const void* ye;          // activation format, rows slot[row * top + k]; null: none
+  const int* slot;
+  const float* w_out;      // [pitch]
+  const float* w_in;       // [pitch], null: no norm behind the sum
+  void* xn;                // [rows][pitch]
+  float* dense;            // optional [rows][width]: x after the sum, without padding
+  const float* embed;      // optional [vocab][pitch]: the row's embedding joins x after that
+  const int* tokens;       // [rows]
+  int vocab;
+};
+
+// Latent projections in fp32 -> normed query latent, and the cached row: normed latent and rotated key part.
+struct LatentPrepArgs {
+  int rows, pitch;         // proj [rows][pitch]: query latent at 0, latent at off_c, rotated part at off_r
+  int q_rank, q_rankp, kv_rank, kv_rankp, rot_dim, rotp, off_c, off_r;
+  const float* proj;
+  const float* q_norm;     // [q_rankp]
+  const float* kv_norm;    // [kv_rankp]
+  float eps;
+  const float2* rot;       // [t_max][pairs] (cos, sin)
+  int pairs;
+  void* cq;                // [rows][q_rankp]
+  void* cache;             // [n_seqs][t_max][kv_rankp + rotp]
+  const int* pos;          // [rows], negative: the row stores nothing
+  const int* seq;          // [rows] cache row, null: row index
+  int t_max, n_seqs, fmt;
+  int* err;
+};
+
 enum : int { PICK_PLAIN = 0, PICK_FIRST = 1, PICK_DECODE = 2 };
 
 struct PickArgs {
@@ -60,6 +96,10 @@ struct PickArgs {
 int arcb_launch_lm_embed(const LmEmbedArgs& a, cudaStream_t stream);
 int arcb_launch_step_begin(const StepState& st, const LmEmbedArgs& a, cudaStream_t stream);
 int arcb_launch_lm_norm(const LmNormArgs& a, cudaStream_t stream);
+int arcb_launch_sandwich_norm(const SandwichArgs& a, cudaStream_t stream);
+int arcb_launch_latent_prep(const LatentPrepArgs& a, cudaStream_t stream);
+// table[p][i] = (cos, sin)(p * base^(-2 i / dims)), i < dims / 2
+int arcb_launch_rot_table(float2* table, int t_max, int dims, double base, cudaStream_t stream);
 int arcb_launch_proj_prep(const ProjArgs& a, const float* proj, cudaStream_t stream);
 int arcb_launch_pick(const PickArgs& a, const StepState& st, cudaStream_t stream);
 int arcb_launch_seg_commit(const StepState& st, const int* seg_seq, const int* seg_pos0, const int* seg_rows, int n,
@@ -69,4 +109,7 @@ int arcb_launch_feed(const StepState& st, const int* seqs, const int* tokens, in
 // container 0 = bfloat16, 1 = half holding the bf16-rounded value, 2 = fp32
 int arcb_launch_pack_blocks(const float* src, void* dst, long long rows, long long cols, int rb, int rbp, int row_off,
                             int cb, int cbp, long long dst_pitch, int container, cudaStream_t stream);
+// the transpose of every head's block: element (h * rb + d, c) goes to row h * rbp + c, column d
+int arcb_launch_pack_heads_t(const float* src, void* dst, int heads, int rb, int rbp, int cols, long long dst_pitch, int container,
+                             cudaStream_t stream);
 void arcb_count_launch(long long n);

@@ -32,7 +32,16 @@ def architectures() -> list[str]:
 
 
 def _import_families() -> None:
-    from . import vodavik  # noqa: F401  (registers itself)
+    from . import logesun, vodavik  # noqa: F401  (they register themselves)
+
+
+def collect_tensors(names: dict, tensors: dict) -> dict:
+    """Checkpoint tensors by (kind, layer); a list of names gives the list of their tensors."""
+    flat = [n for v in names.values() for n in (v if isinstance(v, list) else [v])]
+    missing = sorted(n for n in flat if n not in tensors)
+    if missing:
+        raise ValueError(f"the checkpoint lacks {', '.join(missing[:5])}{' ...' if len(missing) > 5 else ''}")
+    return {key: [tensors[n] for n in v] if isinstance(v, list) else tensors[v] for key, v in names.items()}
 
 
 def build_engine(config: dict, tensors: dict, device="cuda:0", act_format: str = "f16", **options) -> EngineBase:

@@ -10,7 +10,7 @@ keys and values.
 from __future__ import annotations
 
 from .layered import LayeredEngine, LayerSpec, ModelSpec
-from .registry import register
+from .registry import collect_tensors, register
 
 _ATTENTION = {"Q": "q", "Q_B": "q.b", "G": "g", "O": "o", "Q_NORM": "q.norm", "SINK": "sink"}
 _ATTENTION_KV = {"K": "k", "K_B": "k.b", "V": "v", "V_B": "v.b", "K_NORM": "k.norm"}
@@ -66,8 +66,4 @@ def tensor_names(spec: ModelSpec) -> dict[tuple[str, int], str]:
 @register("Vodavik")
 def build(config: dict, tensors: dict, device="cuda:0", act_format: str = "f16", **options) -> LayeredEngine:
     spec = model_spec(config)
-    names = tensor_names(spec)
-    missing = sorted(n for n in names.values() if n not in tensors)
-    if missing:
-        raise ValueError(f"the checkpoint lacks {', '.join(missing[:5])}{' ...' if len(missing) > 5 else ''}")
-    return LayeredEngine(spec, {key: tensors[name] for key, name in names.items()}, device, act_format, **options)
+    return LayeredEngine(spec, collect_tensors(tensor_names(spec), tensors), device, act_format, **options)

@@ -37,7 +37,8 @@ def test_struct_sizes_match_c_layout():
     from mdlarc_scale_b200 import _lib
     assert C.sizeof(_lib.Config) == 14 * 4
     assert C.sizeof(_lib.SessionDesc) == 144  # sizeof(arcb_session_desc) printed by a C compile of the header
-    assert C.sizeof(_lib.PrefillArgs) == 248
+    assert C.sizeof(_lib.PrefillArgs) == 280
+    assert C.sizeof(_lib.LayerDesc) == 120 and C.sizeof(_lib.ModelDesc) == 64
     assert C.sizeof(_lib.PromptBuildArgs) == 160
     assert C.sizeof(_lib.CandidateArgs) == 96
     from mdlarc_scale_b200 import fanout
