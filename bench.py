@@ -9,7 +9,7 @@ for the full 931-token budget over a static KV cache of 1536 positions.  One ste
 the hot path over one such batch: packed prefill + 930 graph-replayed decode steps.  Under
 torchrun every rank runs its own batch (weak scaling, no data-path collective).
 
-`--layered 1280|2048|4096` measures a layered model (Vodavik) beside a TinyTransformer of equal size instead.
+`--layered 1280|2048|4096` measures layered models (Vodavik; `--layered-models logesun,vodavik,tiny`) beside a TinyTransformer of equal size instead.
 
 Prints ONE JSON line (rank 0): generated tokens/s over all GPUs, device-timed (`value`, inputs
 resident in HBM) and end to end through `generate_output` from pinned host tensors (`e2e`),
@@ -321,9 +321,12 @@ def profile_prefill(args):
 # Sizes of the layered-model benchmark: the closest existing model is a TinyTransformer of the same width and
 # depth (heads of 64, its feed-forward sized to the same number of weights).
 LAYERED_SIZES = {
-    "1280": dict(width=1280, heads=20, kv_heads=5, dim=64, vdim=64, ff=5120, tiny_ff=3456),
-    "2048": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, ff=8192, tiny_ff=5440),
-    "4096": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, ff=16384, tiny_ff=10944),
+    "1280": dict(width=1280, heads=20, kv_heads=5, dim=64, vdim=64, ff=5120, tiny_ff=3456,
+                 rot_dim=32, q_rank=768, kv_rank=256, expert_ff=448, shared_ff=1664),
+    "2048": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, ff=8192, tiny_ff=5440,
+                 rot_dim=64, q_rank=1024, kv_rank=512, expert_ff=704, shared_ff=2624),
+    "4096": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, ff=16384, tiny_ff=10944,
+                 rot_dim=64, q_rank=1536, kv_rank=512, expert_ff=1408, shared_ff=5312),
 }
 
 
@@ -370,8 +373,60 @@ def layered_engine(cfg: dict, dev, act_format: str = "f16"):
     return registry.build_engine(cfg, tensors, dev, act_format)
 
 
+def latent_config(size: dict, n_runs: int, window: int, vocab: int = 32000, experts: int = 32, top: int = 4) -> dict:
+    """Latent attention in every layer; gated feed-forwards and mixtures of experts in turn, of the same number of
+    weights per token; two of the layers run twice (``n_runs`` layer runs in all)."""
+    layers = []
+    for n in range(max(2, n_runs - 2)):
+        mixer = {"heads": size["heads"], "dim": size["dim"], "rot_dim": size["rot_dim"], "vdim": size["vdim"], "q_rank": size["q_rank"],
+                 "kv_rank": size["kv_rank"], "mask": {"size": window}, "rot": {"base": 10000.0, "dims": size["rot_dim"]},
+                 "scale": (size["dim"] + size["rot_dim"]) ** -0.5}
+        mlp = {"kind": "dense", "ff": size["tiny_ff"]} if n % 2 == 0 else {
+            "kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": size["expert_ff"], "limit": 7.0},
+            "shared": {"ff": size["shared_ff"], "limit": 7.0}}
+        layers.append({"type": "latent_attention", "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Logesun", "width": size["width"], "vocab": vocab, "layers": layers, "norm": {"eps": 1e-6},
+            "loop": {"start": 0, "stop": 2, "times": 2 if n_runs > 2 else 1}}
+
+
+def latent_engine(cfg: dict, dev, act_format: str = "f16"):
+    """Engine of seeded random weights, drawn on the device."""
+    from mdlarc_scale_b200 import logesun
+    from mdlarc_scale_b200.layered import LayeredEngine
+    spec = logesun.model_spec(cfg)
+    gen = torch.Generator(device=dev).manual_seed(0)
+    width = spec.width
+
+    class Lazy(dict):           # one tensor at a time on the device
+        def items(self):
+            for (kind, n), _ in super().items():
+                s = spec.layers[n]
+                shape = {"EMBED": (spec.vocab, width), "HEAD": (spec.vocab, width), "DQ": (s.q_rank, width), "DQ_NORM": (s.q_rank,),
+                         "UQ": (s.heads * (s.dim + s.rot_dim), s.q_rank), "DKV": (s.kv_rank + s.rot_dim, width), "DKV_NORM": (s.kv_rank,),
+                         "UK": (s.heads * s.dim, s.kv_rank), "UV": (s.heads * s.vdim, s.kv_rank), "SINK": (s.heads,),
+                         "O": (width, s.heads * s.vdim), "GATE": (s.d_ff, width), "UP": (s.d_ff, width), "DOWN": (width, s.d_ff),
+                         "ROUTER": (s.experts, width), "EXPERT_GATE": (s.experts, s.d_ff, width), "EXPERT_UP": (s.experts, s.d_ff, width),
+                         "EXPERT_DOWN": (s.experts, width, s.d_ff), "SHARED_GATE": (s.shared_ff, width), "SHARED_UP": (s.shared_ff, width),
+                         "SHARED_DOWN": (width, s.shared_ff)}.get(kind, (width,))
+                t = torch.randn(shape, generator=gen, device=dev) * (1.0 if kind == "EMBED" else shape[-1] ** -0.5 if len(shape) > 1 else 0.1)
+                yield (kind, n), t + 1.0 if "NORM" in kind else t
+    return LayeredEngine(spec, Lazy(logesun.tensor_names(spec)), dev, act_format)
+
+
+def latent_weights_per_token(spec) -> int:
+    """Weights of the products one token passes, over all layer runs (keys and values counted as expanded)."""
+    total = 0
+    start, stop, times = spec.loop
+    for n, s in enumerate(spec.layers):
+        w = spec.width * (s.q_rank + s.kv_rank + s.rot_dim + s.heads * s.vdim)
+        w += s.heads * ((s.dim + s.rot_dim) * s.q_rank + (s.dim + s.vdim) * s.kv_rank)
+        w += 3 * spec.width * (s.d_ff if s.mlp == "glu" else s.top * s.d_ff + s.shared_ff)
+        total += w * (times if start <= n < stop else 1)
+    return total
+
+
 def bench_layered(args):
-    """Prefill and decode throughput of the Vodavik design (random weights) beside a TinyTransformer of equal
+    """Prefill and decode throughput of the layered designs (random weights) beside a TinyTransformer of equal
     width and depth, same prompts and batch.  Device-timed with CUDA events; every pass streams far more than
     the L2 cache holds."""
     from mdlarc_scale_b200.engine import Engine, chunk_rows, plan_prefill
@@ -394,15 +449,22 @@ def bench_layered(args):
         return e0.elapsed_time(e1) / 1e3 / reps
 
     out = {"benchmark": "layered models", "size": args.layered, "layers": n_layers, "prompts": P, "tokens": T,
-           "decode_batch": B, "decode_context": [T, T + steps], "data": "synthetic", "dtype": "bf16 weights, half operands"}
+           "decode_batch": B, "decode_context": [T, T + steps], "latent_window": args.layered_window, "data": "synthetic",
+           "dtype": "bf16 weights, half operands"}
     sampler = ClockSampler(0)
     with sampler:
         for which in args.layered_models.split(","):
-            if which == "vodavik":
+            layered = which != "tiny"
+            if which == "logesun":
+                eng = latent_engine(latent_config(size, n_layers, args.layered_window), dev)
+                w = latent_weights_per_token(eng.spec)
+                n_attn, heads, dd = eng.spec.n_runs, size["heads"], size["dim"] + size["rot_dim"] + size["vdim"]
+            elif which == "vodavik":
                 eng = layered_engine(layered_config(size, n_layers), dev)
                 w = sum(s.heads * s.dim + s.heads * s.vdim * 2 + (0 if s.mixer == "attention" and s.kv_from >= 0 else
                         s.kv_heads * (s.dim + s.vdim)) + 2 * s.d_ff for s in eng.spec.layers) * eng.spec.width
                 n_attn, heads, dd = sum(s.mixer == "attention" for s in eng.spec.layers), size["heads"], size["dim"] + size["vdim"]
+            if layered:
                 sess = eng.new_session(P, T, 1, P * T, stop_on_end=False)
                 segs = [Segment(i, np.random.default_rng(i).integers(0, 32000, T).tolist()) for i in range(P)]
 
@@ -424,12 +486,14 @@ def bench_layered(args):
                         sess.prefill(p, None)
             t = timed(prefill)
             sess.poll()
-            flop = P * T * 2.0 * w + P * n_attn * heads * dd * float(T) ** 2
+            # pairs of a query and a visible key, twice
+            pairs = float(T) ** 2 - (float(max(0, T - args.layered_window)) ** 2 if which == "logesun" else 0.0)
+            flop = P * T * 2.0 * w + P * n_attn * heads * dd * pairs
             r = {"prefill_tokens_per_s": P * T / t, "prefill_ms": t * 1e3, "prefill_tflops": flop / t / 1e12}
             sess.close()
             # decode: B sequences from a context of T, in prefill calls of bounded size
             per = max(1, 65536 // T)
-            if which == "vodavik":
+            if layered:
                 sess = eng.new_session(B, T + 4 * steps + 8, 4 * steps + 8, per * T, stop_on_end=False)
                 for b in range(0, B, per):
                     sess.prefill_segments([Segment(i, segs[i % P].tokens, arm=True) for i in range(b, min(B, b + per))])
@@ -969,7 +1033,8 @@ def main():
     ap.add_argument("--layered-tokens", type=int, default=2048, help="tokens per prompt and decode context")
     ap.add_argument("--layered-batch", type=int, default=256, help="sequences of a decode step")
     ap.add_argument("--layered-steps", type=int, default=64, help="decode steps per timed pass")
-    ap.add_argument("--layered-models", default="vodavik,tiny")
+    ap.add_argument("--layered-models", default="vodavik,tiny", help="of vodavik, logesun, tiny")
+    ap.add_argument("--layered-window", type=int, default=1024, help="window of the latent attention (logesun)")
     ap.add_argument("--max-new", type=int, default=MAX_NEW,
                     help="tokens generated per sequence (the workload uses 931; smaller only for profiling)")
     args = ap.parse_args()
