@@ -5,12 +5,13 @@
 
 // The queries are already in the latent space: head h of item i scores position p with
 //   (qlat[i][h] . c[p] + qrot[i][h] . r[p]) * scale,   cached row p = [c (kvp columns) | r (rotp columns)],
-// and the output row is the weighted sum of c.
+// and the output row is the weighted sum of c.  A sequence's rows are cut into panels of 64 columns, each panel's rows
+// side by side: whatever reads 64 columns of many rows then reads one piece of memory.
 struct AttnLatentArgs {
   const void* qlat;          // [n_items][H][kvp] activation format
   const void* q;             // rotated part: row i, head h at q + i * H * q_head + h * q_head + q_off
   int q_head, q_off;
-  const void* cache;         // [n_seqs][t_max][kvp + rotp]
+  const void* cache;         // [n_seqs][(kvp + rotp) / 64][t_max][64]
   void* out;                 // [n_items][H][kvp]
   const int* item_seq;       // [n_items] cache row, null = item index
   const int* item_len;       // [n_items] positions [0, len) are cached up to and with the query's own

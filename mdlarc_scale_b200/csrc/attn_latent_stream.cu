@@ -46,7 +46,8 @@ attn_latent_stream_kernel(AttnLatentArgs a) {
 #pragma unroll
   for (int k = 0; k < NV; ++k) acc[k] = make_float4(0.f, 0.f, 0.f, 0.f);
   for (int p = begin + wj; p < len; p += WARPS) {
-    const size_t row = ((size_t)seq * a.t_max + p) * D;
+    const size_t row = ((size_t)seq * (D / 64) * a.t_max + p) * 64;         // of the first panel
+    auto at = [&](int c) { return row + (size_t)(c >> 6) * a.t_max * 64 + (c & 63); };
     float4 v[NV];
     float d = 0.f;
 #pragma unroll
@@ -54,13 +55,13 @@ attn_latent_stream_kernel(AttnLatentArgs a) {
       const int c = lane * 4 + k * 128;
       v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (c < a.kvp) {
-        v[k] = ld_act4(a.cache, row + c, a.fmt);
+        v[k] = ld_act4(a.cache, at(c), a.fmt);
         const float4 q = *reinterpret_cast<const float4*>(s_q + c);
         d += (v[k].x * q.x + v[k].y * q.y) + (v[k].z * q.z + v[k].w * q.w);
       }
     }
     for (int c = a.kvp + lane * 4; c < D; c += 128) {
-      const float4 r = ld_act4(a.cache, row + c, a.fmt);
+      const float4 r = ld_act4(a.cache, at(c), a.fmt);
       const float4 q = *reinterpret_cast<const float4*>(s_q + c);
       d += (r.x * q.x + r.y * q.y) + (r.z * q.z + r.w * q.w);
     }
@@ -123,7 +124,7 @@ cudaError_t launch(const AttnLatentArgs& a, cudaStream_t stream) {
 
 int arcb_launch_attn_latent_stream(const AttnLatentArgs& a, cudaStream_t stream) {
   if (a.n_items <= 0) return 0;
-  if (a.kvp % 4 || a.rotp % 4 || a.q_head % 4 || a.q_off % 4 || (long long)a.n_items * a.n_heads > 0x7fffffffLL) return -1;
+  if (a.kvp % 64 || a.rotp % 64 || a.q_head % 4 || a.q_off % 4 || (long long)a.n_items * a.n_heads > 0x7fffffffLL) return -1;
   cudaError_t e;
   if (a.kvp <= 128) e = launch<1>(a, stream);
   else if (a.kvp <= 256) e = launch<2>(a, stream);

@@ -176,7 +176,7 @@ attn_prefill_gqa_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
         kv_row = (seq * a.n_kv + h / (a.n_heads / a.n_kv)) * a.t_max + key0;
         k_col = v_col = 0;
       }
-      const int rot_row = seq * a.t_max + key0;
+      const int rot_row = (seq * a.rot_panels + a.rot_panel) * a.t_max + key0;
       mbar_expect_tx(b_q, two ? 2 * C::Q_BYTES : C::Q_BYTES);
 #pragma unroll
       for (int c = 0; c < C::QB; ++c) {
@@ -195,7 +195,7 @@ attn_prefill_gqa_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
         for (int c = 0; c < DP / 64; ++c) tma_load_2d(dst + c * BOX_BYTES, &tmap_k, k_col + c * 64, kv_row + j * BKV, b_kfull + 8 * s);
 #pragma unroll
         for (int c = 0; c < DR / 64; ++c)
-          tma_load_2d(dst + (DP / 64 + c) * BOX_BYTES, &tmap_r, a.rot_col + c * 64, rot_row + j * BKV, b_kfull + 8 * s);
+          tma_load_2d(dst + (DP / 64 + c) * BOX_BYTES, &tmap_r, 0, rot_row + c * a.t_max + j * BKV, b_kfull + 8 * s);
         const int t = j % C::V_STAGES;
         if (!mbar_wait_bounded(b_vempty + 8 * t, ((j / C::V_STAGES) & 1) ^ 1)) {
           arcb_set_error(a.err, ARCB_DEV_WAIT_TIMEOUT_MMA);
@@ -489,7 +489,7 @@ int launch(const AttnPrefillGqaArgs& a, cudaStream_t stream) {
   if (r) return 1000 + r;
   CUtensorMap tr = tk;
   if (DR > 0) {
-    r = arcb_make_tmap_2d_16b(&tr, a.k_rot, (uint64_t)a.n_seqs * a.t_max, (uint64_t)a.rot_pitch, BKV, 64, a.act_f16);
+    r = arcb_make_tmap_2d_16b(&tr, a.k_rot, (uint64_t)a.n_seqs * a.rot_panels * a.t_max, 64, BKV, 64, a.act_f16);
     if (r) return 1000 + r;
   }
   const int fmt = a.act_f16 ? 0 : 1;
@@ -510,8 +510,8 @@ bool arcb_attn_prefill_gqa_supported(int dimp, int vdimp, int n_seqs, int n_kv, 
   return scale > 0.f && dimp <= 128 && vdimp <= 128 && (long long)n_seqs * n_kv * t_max < (1ll << 31) - 256;
 }
 
-bool arcb_attn_prefill_latent_supported(int dimp, int rotp, int vdimp, int n_seqs, int t_max, float scale) {
-  return scale > 0.f && dimp <= 128 && rotp == 64 && vdimp <= 128 && (long long)n_seqs * t_max < (1ll << 31) - 256;
+bool arcb_attn_prefill_latent_supported(int dimp, int rotp, int vdimp, int panels, int n_seqs, int t_max, float scale) {
+  return scale > 0.f && dimp <= 128 && rotp == 64 && vdimp <= 128 && (long long)n_seqs * panels * t_max < (1ll << 31) - 256;
 }
 
 int arcb_attn_prefill_gqa_init() {

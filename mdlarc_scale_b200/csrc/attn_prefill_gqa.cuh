@@ -21,19 +21,19 @@ struct AttnPrefillGqaArgs {
   int window;                  // keys [count - window, count) are visible, 0: all [0, count)
   // Expanded keys and values (kv0 set): key / value of position p and head h are columns [h * dimp, ...) and
   // [v_col + h * vdimp, ...) of row kv0[block] + p of a matrix with kv_pitch columns; the last rotp dimensions of
-  // every head's key are columns [rot_col, rot_col + rotp) of row seq * t_max + p of k_rot (rot_pitch columns).
+  // every head's key are row (seq * rot_panels + rot_panel) * t_max + p of k_rot (64 columns).
   const int* kv0;              // [n_qblocks]
   long long kv_rows, kv_pitch;
   int v_col;
   const void* k_rot;
-  int rotp, rot_pitch, rot_col;
+  int rotp, rot_panels, rot_panel;
   float scale;
   int act_f16;
   int* err;
 };
 
 bool arcb_attn_prefill_gqa_supported(int dimp, int vdimp, int n_seqs, int n_kv, int t_max, float scale);
-bool arcb_attn_prefill_latent_supported(int dimp, int rotp, int vdimp, int n_seqs, int t_max, float scale);
+bool arcb_attn_prefill_latent_supported(int dimp, int rotp, int vdimp, int panels, int n_seqs, int t_max, float scale);
 int arcb_attn_prefill_gqa_init();
 int arcb_launch_attn_prefill_gqa(const AttnPrefillGqaArgs& a, cudaStream_t stream);
 void arcb_count_launch(long long n);

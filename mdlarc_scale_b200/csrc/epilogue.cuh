@@ -33,6 +33,8 @@ struct GluArgs {
 // Products whose rows or columns belong to groups.  All fields zero: one plain product.
 //   rows    : tile_src[t] is the A row of output rows [128 t, 128 t + 128) (null: 128 t); tile_group[t] picks the
 //             rows [group * group_rows, ...) of W; n_tiles (device) is the number of tiles that hold anything
+//   panels  : A is cut into panels of 64 columns, [sequence][panels][panel_rows][64]; tile_src then counts rows as
+//             sequence * panel_rows + row
 //   columns : columns [c n_group, (c + 1) n_group) read A columns [c a_group, c a_group + K)
 struct GroupArgs {
   const int* tile_src;
@@ -42,7 +44,8 @@ struct GroupArgs {
   long long w_rows;      // rows of W in all groups
   int n_group, a_group;
   int lda;               // row pitch of A in elements, 0: K
-  long long a_rows;      // rows of A, 0: M
+  long long a_rows;      // rows of A, 0: M (panels: of all panels)
+  int panels, panel_rows;
 };
 
 // Fused projection of a mixer: the output columns are sections of whole heads, every head padded to
@@ -314,6 +317,13 @@ __device__ __forceinline__ void epi_swiglu_quad(const GemmEpilogue& e, int m, in
   pk.x = pack2_act_chk(silu_f(g.x) * u.x, silu_f(g.y) * u.y, e.act_f16, e.err);
   pk.y = pack2_act_chk(silu_f(g.z) * u.z, silu_f(g.w) * u.w, e.act_f16, e.err);
   *reinterpret_cast<uint2*>(reinterpret_cast<uint16_t*>(e.out16) + (size_t)m * (e.N >> 1) + j) = pk;
+}
+
+// first A row of a row tile
+__device__ __forceinline__ int group_a_row(const GroupArgs& g, int tile) {
+  if (!g.tile_src) return tile * 128;
+  const int r = g.tile_src[tile];
+  return g.panels ? r + r / g.panel_rows * (g.panels - 1) * g.panel_rows : r;
 }
 
 // ---- EPI_ACT ----

@@ -608,7 +608,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
       bool ok = true;
       for (int tile = blockIdx.x; ok && tile < tiles_total; tile += gridDim.x) {
         const int m_blk = tile / tiles_n, n_blk = tile - m_blk * tiles_n;
-        const int a_row = g.tile_src ? g.tile_src[m_blk] : m_blk * TC_BM;
+        const int a_row = group_a_row(g, m_blk);
         const int w_row = n_blk * BN + (g.tile_group ? g.tile_group[m_blk] * g.group_rows : 0);
         const int a_col = g.n_group ? n_blk * BN / g.n_group * g.a_group : 0;
         for (int kb = 0; kb < num_k; ++kb, ++kbt) {
@@ -624,7 +624,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
           const uint32_t full = bar_base + 8 * s;
           const uint32_t a_dst = base + s * Cfg::STAGE_BYTES;
           mbar_expect_tx(full, Cfg::STAGE_BYTES);
-          tma_load_2d(a_dst, &tmap_a, a_col + kb * TC_BK, a_row, full);
+          if (g.panels) tma_load_2d(a_dst, &tmap_a, 0, a_row + kb * g.panel_rows, full);
+          else tma_load_2d(a_dst, &tmap_a, a_col + kb * TC_BK, a_row, full);
           tma_load_2d(a_dst + Cfg::A_BYTES, &tmap_b, kb * TC_BK, w_row, full);
         }
       }
@@ -825,7 +826,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constan
       for (int tile = pair; ok && tile < tiles_total; tile += n_pairs) {
         const int m_blk = tile / tiles_n, n_blk = tile - m_blk * tiles_n;
         const int m_tile = 2 * m_blk + (int)rank;
-        const int a_row = g.tile_src ? g.tile_src[m_tile] : m_tile * 128;
+        const int a_row = group_a_row(g, m_tile);
         const int w_row = n_blk * BN + (int)rank * 128 + (g.tile_group ? g.tile_group[m_tile] * g.group_rows : 0);
         for (int kb = 0; kb < num_k; ++kb, ++kbt) {
           const int s = kbt % Cfg::STAGES;
@@ -840,7 +841,8 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constan
           const uint32_t full = bar_base + 8 * s;
           const uint32_t a_dst = base + s * Cfg::STAGE_BYTES;
           if (rank == 0) mbar_expect_tx(full, 2 * Cfg::STAGE_BYTES);  // both CTAs' bytes land on CTA 0's barrier
-          tma_load_2d_2cta(a_dst, &tmap_a, kb * TC_BK, a_row, full);
+          if (g.panels) tma_load_2d_2cta(a_dst, &tmap_a, 0, a_row + kb * g.panel_rows, full);
+          else tma_load_2d_2cta(a_dst, &tmap_a, kb * TC_BK, a_row, full);
           tma_load_2d_2cta(a_dst + Cfg::A_BYTES, &tmap_b, kb * TC_BK, w_row, full);
         }
       }
@@ -1497,7 +1499,9 @@ static int launch_gemm_mode(const void* a16, const void* w16, const GemmEpilogue
                             int act_f16, bool use_tc, int tc_variant, cudaStream_t stream) {
   const int M = ep.M, N = ep.N;
   const GroupArgs& g = ep.grp;
-  const uint64_t a_rows = g.a_rows ? (uint64_t)g.a_rows : (uint64_t)M, a_cols = g.lda ? (uint64_t)g.lda : (uint64_t)K;
+  const uint64_t a_rows = g.a_rows ? (uint64_t)g.a_rows : (uint64_t)M;
+  const uint64_t a_cols = g.panels ? 64 : g.lda ? (uint64_t)g.lda : (uint64_t)K;
+  if (g.panels && (!use_tc || g.n_group || !g.tile_src || !g.a_rows)) return -1;
   const uint64_t w_rows = g.w_rows ? (uint64_t)g.w_rows : (uint64_t)N;
   if (use_tc) {
     if constexpr (MODE == EPI_ACT) {

@@ -44,6 +44,7 @@ struct LmLayer {
   float* norm2b = nullptr;
   // latent attention
   int hp = 0;                  // heads, one zero head added where sections would not fill whole column tiles
+  int panels() const { return (kvp + rotp) / 64; }   // of the cached rows
   int q_rankp = 0, kvp = 0, rotp = 0, n_down = 0, n_expand = 0, rot_table = 0;
   void* w_uq = nullptr;        // [hp * (dimp + rotp)][q_rankp]; w_proj holds [n_down][Wp]: query latent, latent, rotated part
   void* w_ukv = nullptr;       // [n_expand][kvp]: keys of all heads, then values of all heads
@@ -152,7 +153,7 @@ bool lm_tc(const LayeredModel& m) { return m.fmt != 2 && m.d.gemm_path != ARCB_G
 // keys and values expanded for the tensor-core prefill attention
 bool lm_expands(const LayeredModel& m, const LmLayer& L, int B, int T) {
   return L.d.mixer == ARCB_MIXER_LATENT && lm_tc(m) && m.d.attn_path == ARCB_ATTN_AUTO &&
-         arcb_attn_prefill_latent_supported(L.dimp, L.rotp, L.vdimp, B, T, L.d.scale);
+         arcb_attn_prefill_latent_supported(L.dimp, L.rotp, L.vdimp, L.panels(), B, T, L.d.scale);
 }
 // Rows of the expansion scratch: enough for a block of queries with its window, and for about 16 k keys (more of
 // them leave the L2 cache before they are read).
@@ -794,14 +795,14 @@ int lm_latent(arcb_session* s, int l, const Rows& R, cudaStream_t stream) {
       if (nt * 128 > ls->expand_rows) return arcb_fail(ARCB_E_ARG, "a group exceeds the expansion scratch");
       GemmEpilogue ek{};
       ek.mode = EPI_ACT; ek.M = nt * 128; ek.N = L.n_expand; ek.out16 = ls->expand; ek.act_f16 = m.fmt; ek.err = s->eng->d_err;
-      ek.grp.tile_src = pa.d_tile_src + t0; ek.grp.lda = L.kvp + L.rotp; ek.grp.a_rows = (long long)B * T;
+      ek.grp.tile_src = pa.d_tile_src + t0; ek.grp.panels = L.panels(); ek.grp.panel_rows = T; ek.grp.a_rows = (long long)B * L.panels() * T;
       CKL(lm_gemm(m, ls->k[l], L.w_ukv, ek, L.kvp, stream), "expansion gemm");
       AttnPrefillGqaArgs a{};
       a.q = ls->proj; a.q_pitch = L.n_proj; a.k = ls->expand; a.v = ls->expand; a.out = ls->mix; a.seq = R.seq; a.kv_count = R.kv_len;
       a.qblock_row0 = pa.d_qblock_row0 + q0; a.qblock_rows = pa.d_qblock_rows + q0; a.kv0 = pa.d_qblock_kv0 + q0; a.n_qblocks = nq;
       a.sink = d.sink ? L.sink : nullptr; a.n_rows = R.n; a.n_heads = a.n_kv = L.hp; a.dimp = L.dimp; a.vdimp = L.vdimp; a.t_max = T;
       a.n_seqs = B; a.window = d.window; a.kv_rows = nt * 128; a.kv_pitch = L.n_expand; a.v_col = L.hp * L.dimp; a.k_rot = ls->k[l];
-      a.rotp = L.rotp; a.rot_pitch = L.kvp + L.rotp; a.rot_col = L.kvp; a.scale = d.scale; a.act_f16 = m.fmt; a.err = s->eng->d_err;
+      a.rotp = L.rotp; a.rot_panels = L.panels(); a.rot_panel = L.kvp / 64; a.scale = d.scale; a.act_f16 = m.fmt; a.err = s->eng->d_err;
       CKL(arcb_launch_attn_prefill_gqa(a, stream), "prefill attention");
     }
   } else {

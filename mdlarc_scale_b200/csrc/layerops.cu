@@ -285,8 +285,8 @@ latent_prep_kernel(LatentPrepArgs a) {
     if (tid == 0) arcb_set_error(a.err, ARCB_DEV_BAD_INDEX);
     return;
   }
-  const size_t at = ((size_t)seq * a.t_max + pos) * (a.kv_rankp + a.rotp);
-  for (int i = tid * 4; i < a.kv_rankp; i += STEP) st_act4(a.cache, at + i, normed(p + a.off_c, a.kv_norm, i, ic), a.fmt);
+  auto at = [&](int c) { return (((size_t)seq * ((a.kv_rankp + a.rotp) >> 6) + (c >> 6)) * a.t_max + pos) * 64 + (c & 63); };
+  for (int i = tid * 4; i < a.kv_rankp; i += STEP) st_act4(a.cache, at(i), normed(p + a.off_c, a.kv_norm, i, ic), a.fmt);
   for (int i = tid * 4; i < a.rotp; i += STEP) {
     const float4 v = *reinterpret_cast<const float4*>(p + a.off_r + i);
     float4 o = v;
@@ -301,7 +301,7 @@ latent_prep_kernel(LatentPrepArgs a) {
       o.z = v.z * c.x - v.w * c.y;
       o.w = v.w * c.x + v.z * c.y;
     }
-    st_act4(a.cache, at + a.kv_rankp + i, o, a.fmt);
+    st_act4(a.cache, at(a.kv_rankp + i), o, a.fmt);
   }
 }
 
@@ -632,7 +632,7 @@ int arcb_launch_sandwich_norm(const SandwichArgs& a, cudaStream_t stream) {
 
 int arcb_launch_latent_prep(const LatentPrepArgs& a, cudaStream_t stream) {
   if (a.rows <= 0) return 0;
-  if (a.q_rankp % 4 || a.kv_rankp % 4 || a.rotp % 4 || a.off_c % 4 || a.off_r % 4 || a.pitch % 4) return -1;
+  if (a.q_rankp % 4 || a.kv_rankp % 64 || a.rotp % 64 || a.off_c % 4 || a.off_r % 4 || a.pitch % 4) return -1;
   const cudaError_t e = arcb_launch(latent_prep_kernel<4>, dim3(a.rows), dim3(128), 0, stream, a);
   arcb_count_launch(1);
   return (int)e;

@@ -75,7 +75,7 @@ struct LatentPrepArgs {
   const float2* rot;       // [t_max][pairs] (cos, sin)
   int pairs;
   void* cq;                // [rows][q_rankp]
-  void* cache;             // [n_seqs][t_max][kv_rankp + rotp]
+  void* cache;             // [n_seqs][(kv_rankp + rotp) / 64][t_max][64]
   const int* pos;          // [rows], negative: the row stores nothing
   const int* seq;          // [rows] cache row, null: row index
   int t_max, n_seqs, fmt;
