@@ -16,7 +16,8 @@ enum : int {
 };
 
 // Rotation of neighbouring column pairs of every head: head h owns columns [h * head, (h + 1) * head), its
-// columns off + 2 i and off + 2 i + 1 (i < pairs) turn by the angle whose (cos, sin) is table[pos][i].
+// columns off + 2 i and off + 2 i + 1 (i < pairs) turn by the angle whose (cos, sin) is table[pos][i].  pairs covers
+// all columns from off to the head's end; pairs that do not turn hold (1, 0).
 struct RotArgs {
   const float2* table;   // [t_max][pairs], null: nothing turns
   const int* pos;        // [M], negative: position 0
@@ -332,23 +333,15 @@ __device__ __forceinline__ const float2* rot_row(const GemmEpilogue& e, int m) {
   const int p = min(max(e.rot.pos[m], 0), e.rot.t_max - 1);
   return e.rot.table + (size_t)p * e.rot.pairs;
 }
+// two neighbouring pairs by (cos, sin, cos, sin)
+__device__ __forceinline__ float4 rotate4(float4 v, float4 a) {
+  return make_float4(v.x * a.x - v.y * a.y, v.y * a.x + v.x * a.y, v.z * a.z - v.w * a.w, v.w * a.z + v.z * a.w);
+}
 // columns n .. n + 3 (n % 4 == 0) of a row whose table row is cs
 __device__ __forceinline__ float4 rot_quad(const GemmEpilogue& e, const float2* cs, int n, float4 v) {
   const int c = n % e.rot.head - e.rot.off;
   if (c < 0) return v;
-  const int i = c >> 1;
-  float4 o = v;
-  if (i < e.rot.pairs) {
-    const float2 a = __ldg(cs + i);
-    o.x = v.x * a.x - v.y * a.y;
-    o.y = v.y * a.x + v.x * a.y;
-  }
-  if (i + 1 < e.rot.pairs) {
-    const float2 a = __ldg(cs + i + 1);
-    o.z = v.z * a.x - v.w * a.y;
-    o.w = v.w * a.x + v.z * a.y;
-  }
-  return o;
+  return rotate4(v, __ldg(reinterpret_cast<const float4*>(cs + (c >> 1))));
 }
 __device__ __forceinline__ void epi_act_quad(const GemmEpilogue& e, int m, int n, float4 v) {
   if (e.rot.table) v = rot_quad(e, rot_row(e, m), n, v);

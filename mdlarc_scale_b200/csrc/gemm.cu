@@ -214,18 +214,23 @@ __device__ __forceinline__ void epilogue_act_tma(const GemmEpilogue& ep, const C
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
       uint32_t r[32];
+      float4 a[8];
+      if (in_rot >= 0) {
+        const float4* src = reinterpret_cast<const float4*>(cs + ((in_rot + half * 32) >> 1));
+#pragma unroll
+        for (int i = 0; i < 8; ++i) a[i] = __ldg(src + i);
+      }
       tmem_ld_32x32(t_row + b * 64 + half * 32, r);
       tmem_wait_ld();
       if (in_rot >= 0) {
-        const int i0 = (in_rot + half * 32) >> 1;
 #pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          if (i0 + i < ep.rot.pairs) {
-            const float2 a = __ldg(cs + i0 + i);
-            const float x = __uint_as_float(r[2 * i]), y = __uint_as_float(r[2 * i + 1]);
-            r[2 * i] = __float_as_uint(x * a.x - y * a.y);
-            r[2 * i + 1] = __float_as_uint(y * a.x + x * a.y);
-          }
+        for (int i = 0; i < 8; ++i) {
+          const float4 v = rotate4(make_float4(__uint_as_float(r[4 * i]), __uint_as_float(r[4 * i + 1]), __uint_as_float(r[4 * i + 2]),
+                                               __uint_as_float(r[4 * i + 3])), a[i]);
+          r[4 * i] = __float_as_uint(v.x);
+          r[4 * i + 1] = __float_as_uint(v.y);
+          r[4 * i + 2] = __float_as_uint(v.z);
+          r[4 * i + 3] = __float_as_uint(v.w);
         }
       }
 #pragma unroll

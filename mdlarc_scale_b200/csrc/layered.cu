@@ -67,7 +67,7 @@ struct LmRun {
 };
 
 struct RotTable {
-  int dims;
+  int dims, pairs;
   double base;
 };
 
@@ -131,7 +131,8 @@ struct LmWs {
   int head_rows, lat_rows, max_slots, max_rt;
 };
 
-constexpr int MOE_FIXED_INTS = 2 * MOE_MAX_EXPERTS + 64;   // counts, offsets, number of tiles
+// counts of every layer run with routed experts, and the number of tiles
+size_t moe_ints(const LayeredModel& m) { return m.has_moe ? m.runs.size() * MOE_MAX_EXPERTS + 64 : 0; }
 
 // Feed-forwards that go through the routed experts' buffers: the most slots and (row, choice) pairs of `rows` rows.
 void moe_sizes(const LayeredModel& m, int rows, int* slots, int* rt, int* ffp, int* zp) {
@@ -216,7 +217,7 @@ LmWs lm_ws(const LayeredModel& m, int B, int P, int splits, int requested) {
     }
   w.ascratch = take(asz);
   w.gscratch = take(align_up((size_t)B, 128) * m.n_wide_max * 4);
-  w.n_ints = (size_t)B * 7 + 64 + (m.has_moe ? MOE_FIXED_INTS : 0);
+  w.n_ints = (size_t)B * 7 + 64 + moe_ints(m);
   w.ints = take(w.n_ints * 4);
   w.y = take(m.sandwich() ? R * m.wp * 4 : 0);
   w.cq = take(R * (size_t)m.cq_max * m.es);
@@ -242,7 +243,7 @@ size_t kv_plane(const LayeredModel& m, const LmLayer& L, int B, int T, bool valu
 size_t latent_plane(const LayeredModel& m, const LmLayer& L, int B, int T) {
   return align_up((size_t)B * T * (L.kvp + L.rotp) * m.es, 1024);
 }
-size_t rot_plane(const RotTable& r, int T) { return align_up((size_t)T * (r.dims / 2) * sizeof(float2), 1024); }
+size_t rot_plane(const RotTable& r, int T) { return align_up((size_t)T * r.pairs * sizeof(float2), 1024); }
 size_t expand_plane(const LayeredModel& m, int B, int T) {
   return align_up((size_t)lm_expand_rows(m, B, T) * m.expand_max * m.es, 1024);
 }
@@ -276,7 +277,8 @@ extern "C" int arcb_engine_create_layered(const arcb_model_desc* md, const arcb_
       if (d.q_rank <= 0 || d.kv_rank <= 0 || d.rot_dim < 0 || d.rot_dims < 0 || d.rot_dims > d.rot_dim || d.rot_dims % 2)
         return arcb_fail(ARCB_E_ARG, "bad latent sizes");
       if (d.rot_dims > 0 && !(d.rot_base > 0.)) return arcb_fail(ARCB_E_ARG, "rot_base must be positive");
-      if (d.kv_rank > 2048) return arcb_fail(ARCB_E_UNSUPPORTED, "latents above 2048 are not implemented");
+      if (d.kv_rank > 2048 || pad64(d.q_rank) + pad128(d.kv_rank) + pad64(d.rot_dim) > 6144)
+        return arcb_fail(ARCB_E_UNSUPPORTED, "latents above 2048, or above 6144 columns with the query latent, are not implemented");
       if (d.qkv_bias || d.qk_norm || d.out_gate || d.q_temp_every || d.kv_from >= 0)
         return arcb_fail(ARCB_E_UNSUPPORTED, "latent attention has no biases, head norms, output gate, query gain or shared cache");
     } else if (d.dim > 256 || d.vdim > 256) {
@@ -350,10 +352,10 @@ extern "C" int arcb_engine_create_layered(const arcb_model_desc* md, const arcb_
       L.rot_table = -1;
       if (d.rot_dims > 0) {
         for (size_t i = 0; i < m->rots.size(); ++i)
-          if (m->rots[i].dims == d.rot_dims && m->rots[i].base == d.rot_base) L.rot_table = (int)i;
+          if (m->rots[i].dims == d.rot_dims && m->rots[i].pairs == L.rotp / 2 && m->rots[i].base == d.rot_base) L.rot_table = (int)i;
         if (L.rot_table < 0) {
           L.rot_table = (int)m->rots.size();
-          m->rots.push_back({d.rot_dims, d.rot_base});
+          m->rots.push_back({d.rot_dims, L.rotp / 2, d.rot_base});
         }
       }
       const bool sees_all = d.window == 0 || (m->cq_max > 0 && m->window_max == 0);
@@ -677,8 +679,7 @@ int lm_session_create(arcb_session* s) {
   st.kv_len = p + 5 * B; st.finished = p + 6 * B; st.n_finished = p + 7 * B;
   if (m.has_moe) {
     mo.count = p + 7 * B + 64;
-    mo.offset = mo.count + MOE_MAX_EXPERTS;
-    mo.n_tiles = mo.offset + MOE_MAX_EXPERTS;
+    mo.n_tiles = mo.count + m.runs.size() * MOE_MAX_EXPERTS;
   }
   st.out_tokens = d.d_out_tokens; st.forced = d.d_forced; st.step_logits = d.d_step_logits;
   st.temperature = d.temperature; st.top_k = d.top_k; st.sample_seed = d.sample_seed; st.sample_stream = d.d_sample_stream;
@@ -780,12 +781,12 @@ int lm_latent(arcb_session* s, int l, const Rows& R, cudaStream_t stream) {
   LatentPrepArgs p{};
   p.rows = R.n; p.pitch = L.n_down; p.q_rank = d.q_rank; p.q_rankp = L.q_rankp; p.kv_rank = d.kv_rank; p.kv_rankp = L.kvp;
   p.rot_dim = d.rot_dim; p.rotp = L.rotp; p.off_c = L.q_rankp; p.off_r = L.q_rankp + L.kvp; p.proj = ls->proj32;
-  p.q_norm = L.dq_norm; p.kv_norm = L.dkv_norm; p.eps = m.d.norm_eps; p.rot = rot; p.pairs = rot ? d.rot_dims / 2 : 0;
+  p.q_norm = L.dq_norm; p.kv_norm = L.dkv_norm; p.eps = m.d.norm_eps; p.rot = rot;
   p.cq = ls->cq; p.cache = ls->k[l]; p.pos = R.pos; p.seq = R.seq; p.t_max = T; p.n_seqs = B; p.fmt = m.fmt; p.err = s->eng->d_err;
   CKL(arcb_launch_latent_prep(p, stream), "latent prep");
   GemmEpilogue eq{};
   eq.mode = EPI_ACT; eq.M = R.n; eq.N = L.n_proj; eq.out16 = ls->proj; eq.act_f16 = m.fmt; eq.err = s->eng->d_err;
-  if (rot) eq.rot = RotArgs{rot, R.pos, d.rot_dims / 2, qh, L.dimp, T};
+  if (rot) eq.rot = RotArgs{rot, R.pos, L.rotp / 2, qh, L.dimp, T};
   CKL(lm_gemm(m, ls->cq, L.w_uq, eq, L.q_rankp, stream), "query gemm");
 
   if (R.pa && R.pa->n_groups > 0 && lm_expands(m, L, B, T)) {
@@ -834,10 +835,11 @@ int lm_latent(arcb_session* s, int l, const Rows& R, cudaStream_t stream) {
   return lm_residual(s, ls->mix, L.w_out, L.k_out, R.n, R.pa == nullptr, stream);
 }
 
-// Feed-forward of layer L from xn.  Routed experts leave their rows in ls->moe_out (joined by the norm that follows).
-int lm_mlp(arcb_session* s, const LmLayer& L, const Rows& R, cudaStream_t stream) {
+// Feed-forward of layer run l from xn.  Routed experts leave their rows in ls->moe_out (joined by the norm that follows).
+int lm_mlp(arcb_session* s, int l, const Rows& R, cudaStream_t stream) {
   const LayeredModel& m = *s->eng->lm;
   LayeredSession* ls = s->ls;
+  const LmLayer& L = m.layers[m.runs[l].layer];
   const arcb_layer_desc& d = L.d;
   const bool step = R.pa == nullptr;
   GemmEpilogue eu{};
@@ -854,9 +856,15 @@ int lm_mlp(arcb_session* s, const LmLayer& L, const Rows& R, cudaStream_t stream
     CKL(lm_gemm(m, ls->xn, L.w_up, eu, m.wp, stream), "gate/up gemm");
     return lm_residual(s, ls->hid, L.w_down, L.ffp, R.n, step, stream);
   }
-  int r = lm_store32(s, ls->xn, L.w_router, m.wp, L.n_router, R.n, const_cast<float*>(ls->moe.z), false, stream);
-  if (r) return r;
   MoeArgs mo = ls->moe;
+  mo.count += (size_t)l * MOE_MAX_EXPERTS;
+  if (arcb_moe_router_inside(R.n, d.experts, m.wp, m.fmt)) {
+    mo.z = nullptr;
+    mo.w_router = L.w_router;
+  } else {
+    const int r = lm_store32(s, ls->xn, L.w_router, m.wp, L.n_router, R.n, const_cast<float*>(mo.z), false, stream);
+    if (r) return r;
+  }
   mo.rows = R.n; mo.experts = d.experts; mo.top = d.top; mo.z_pitch = L.n_router; mo.xn = ls->xn; mo.pitch = m.wp; mo.fmt = m.fmt;
   // pairs of row tiles (one expert each) once an expert fills them on average
   mo.gran = lm_tc(m) && arcb_gemm_max_pairs() > 0 && (long long)R.n * d.top >= 256ll * d.experts ? 256 : 128;
@@ -976,7 +984,7 @@ int lm_layers_sandwich(arcb_session* s, const Rows& R, float* residuals, cudaStr
     else last();
     CKL(arcb_launch_sandwich_norm(a, stream), "norm");
     if (!L.ffp) continue;
-    r = lm_mlp(s, L, R, stream);
+    r = lm_mlp(s, l, R, stream);
     if (r) return r;
     a.w_out = L.norm2b;
     if (L.d.mlp == ARCB_MLP_MOE) {
@@ -1002,7 +1010,7 @@ int lm_layers(arcb_session* s, const Rows& R, float* residuals, cudaStream_t str
     r = lm_norm(s, L.norm1, R.n, last && !L.ffp ? 1.f : m.d.residual_alpha, L.ffp ? nullptr : dense, stream);
     if (r) return r;
     if (L.ffp) {
-      r = lm_mlp(s, L, R, stream);
+      r = lm_mlp(s, l, R, stream);
       if (!r) r = lm_norm(s, L.norm2, R.n, last ? 1.f : m.d.residual_alpha, dense, stream);
       if (r) return r;
     }
@@ -1038,7 +1046,8 @@ LmEmbedArgs lm_embed_args(const arcb_session* s, int rows, const int* tokens) {
   const LayeredModel& m = *s->eng->lm;
   LmEmbedArgs a{};
   a.rows = rows; a.width = m.d.width; a.pitch = m.wp; a.vocab = m.d.vocab; a.fmt = m.fmt; a.token_ids = tokens;
-  a.embed = m.embed; a.alpha = m.d.residual_alpha; a.x = s->ls->x; a.xn = s->ls->xn;
+  a.embed = m.embed; a.alpha = m.d.residual_alpha; a.x = s->ls->x; a.xn = m.sandwich() ? nullptr : s->ls->xn;
+  a.zero = s->ls->moe.count; a.n_zero = m.has_moe ? (int)(m.runs.size() * MOE_MAX_EXPERTS) : 0;
   return a;
 }
 
@@ -1051,7 +1060,7 @@ int lm_clear(arcb_session* s, cudaStream_t stream) {
   CK(cudaMemsetAsync(s->desc.d_kv_cache, 0, (size_t)lm_cache_bytes(s->eng, s->desc.n_seqs, s->desc.t_max), stream));
   const LayeredModel& m = *s->eng->lm;
   for (size_t i = 0; i < m.rots.size(); ++i)
-    CKL(arcb_launch_rot_table(ls->rot[i], s->desc.t_max, m.rots[i].dims, m.rots[i].base, stream), "rotation table");
+    CKL(arcb_launch_rot_table(ls->rot[i], s->desc.t_max, m.rots[i].pairs, m.rots[i].dims, m.rots[i].base, stream), "rotation table");
   ls->cleared = true;
   return ARCB_OK;
 }

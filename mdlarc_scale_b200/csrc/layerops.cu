@@ -20,15 +20,21 @@ __device__ __forceinline__ void embed_row(const LmEmbedArgs& a, int row, int tok
   float* x = a.x + (size_t)row * a.pitch;
   for (int i = lane * 4; i < a.pitch; i += 128) {   // the table's padding columns are zero
     const float4 v = __ldg(reinterpret_cast<const float4*>(src + i));
-    st_act4(a.xn, (size_t)row * a.pitch + i, v, a.fmt);
+    if (a.xn) st_act4(a.xn, (size_t)row * a.pitch + i, v, a.fmt);
     *reinterpret_cast<float4*>(x + i) = make_float4(a.alpha * v.x, a.alpha * v.y, a.alpha * v.z, a.alpha * v.w);
   }
+}
+
+__device__ __forceinline__ void embed_zero(const LmEmbedArgs& a) {
+  if (blockIdx.x == 0)
+    for (int i = threadIdx.x; i < a.n_zero; i += blockDim.x) a.zero[i] = 0;
 }
 
 __global__ void __launch_bounds__(ROWS_PER_CTA * 32)
 lm_embed_kernel(LmEmbedArgs a) {
   pdl_launch_dependents();
   pdl_wait();
+  embed_zero(a);
   const int row = blockIdx.x * ROWS_PER_CTA + (threadIdx.x >> 5);
   if (row >= a.rows) return;
   embed_row(a, row, a.token_ids[row], threadIdx.x & 31);
@@ -38,6 +44,7 @@ __global__ void __launch_bounds__(ROWS_PER_CTA * 32)
 step_begin_kernel(StepState st, LmEmbedArgs a) {
   pdl_launch_dependents();
   pdl_wait();
+  embed_zero(a);
   const int b = blockIdx.x * ROWS_PER_CTA + (threadIdx.x >> 5);
   if (b >= st.n_seqs) return;
   const int lane = threadIdx.x & 31;
@@ -187,9 +194,8 @@ sandwich_norm_kernel(SandwichArgs a) {
       }
     return v;
   };
-  auto added = [&](int i, float4 v, float inv) {
+  auto added = [&](int i, float4 r, float4 v, float inv) {
     const float4 g = __ldg(reinterpret_cast<const float4*>(a.w_out + i));
-    const float4 r = *reinterpret_cast<const float4*>(x + i);
     return make_float4(r.x + (v.x * inv) * g.x, r.y + (v.y * inv) * g.y, r.z + (v.z * inv) * g.z, r.w + (v.w * inv) * g.w);
   };
   auto dense = [&](int i, float4 v) {
@@ -213,12 +219,16 @@ sandwich_norm_kernel(SandwichArgs a) {
   };
   // padding columns are zero in y, x, the embedding and the gains
   if constexpr (REGS) {
-    float4 v[NV];
+    float4 v[NV], r[NV];
     float ss = 0.f;
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
       const int i = (tid + k * 128) * 4;
-      v[k] = i < a.pitch ? sublayer(i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      v[k] = r[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < a.pitch) {
+        v[k] = sublayer(i);
+        r[k] = *reinterpret_cast<const float4*>(x + i);
+      }
       ss += sum_sq(v[k]);
     }
     float inv = 1.f / sqrtf(cta_sum<4>(ss, sm[0]) * inv_n + a.eps);
@@ -227,7 +237,7 @@ sandwich_norm_kernel(SandwichArgs a) {
     for (int k = 0; k < NV; ++k) {
       const int i = (tid + k * 128) * 4;
       if (i >= a.pitch) continue;
-      v[k] = added(i, v[k], inv);
+      v[k] = added(i, r[k], v[k], inv);
       if (a.dense) dense(i, v[k]);
       v[k] = with_embed(i, v[k]);
       *reinterpret_cast<float4*>(x + i) = v[k];
@@ -246,7 +256,7 @@ sandwich_norm_kernel(SandwichArgs a) {
     float inv = 1.f / sqrtf(cta_sum<4>(ss, sm[0]) * inv_n + a.eps);
     ss = 0.f;
     for (int i = tid * 4; i < a.pitch; i += 512) {
-      float4 v = added(i, sublayer(i), inv);
+      float4 v = added(i, *reinterpret_cast<const float4*>(x + i), sublayer(i), inv);
       if (a.dense) dense(i, v);
       v = with_embed(i, v);
       *reinterpret_cast<float4*>(x + i) = v;
@@ -258,50 +268,60 @@ sandwich_norm_kernel(SandwichArgs a) {
   }
 }
 
-// One CTA per row, WARPS warps; both norms' sums in one pass, then the row is read again (L1).
-template <int WARPS>
-__global__ void __launch_bounds__(WARPS * 32)
+// One CTA of four warps per row; NV float4 per thread hold the whole row of projections, both norms' sums are taken in
+// one exchange.
+template <int NV>
+__global__ void __launch_bounds__(128)
 latent_prep_kernel(LatentPrepArgs a) {
   pdl_launch_dependents();
   pdl_wait();
-  __shared__ float sm[2][WARPS];
-  constexpr int STEP = WARPS * 32 * 4;
+  __shared__ float2 sm[4];
   const int row = blockIdx.x, tid = threadIdx.x;
-  const float* p = a.proj + (size_t)row * a.pitch;
-  float sq = 0.f, sc = 0.f;
-  for (int i = tid * 4; i < a.q_rankp; i += STEP) sq += sum_sq(*reinterpret_cast<const float4*>(p + i));
-  for (int i = tid * 4; i < a.kv_rankp; i += STEP) sc += sum_sq(*reinterpret_cast<const float4*>(p + a.off_c + i));
-  const float iq = 1.f / sqrtf(cta_sum<WARPS>(sq, sm[0]) / (float)a.q_rank + a.eps);
-  const float ic = 1.f / sqrtf(cta_sum<WARPS>(sc, sm[1]) / (float)a.kv_rank + a.eps);
-  auto normed = [&](const float* src, const float* w, int i, float inv) {
-    const float4 v = *reinterpret_cast<const float4*>(src + i), g = __ldg(reinterpret_cast<const float4*>(w + i));
-    return make_float4((v.x * inv) * g.x, (v.y * inv) * g.y, (v.z * inv) * g.z, (v.w * inv) * g.w);
-  };
-  for (int i = tid * 4; i < a.q_rankp; i += STEP)
-    st_act4(a.cq, (size_t)row * a.q_rankp + i, normed(p, a.q_norm, i, iq), a.fmt);
   const int pos = a.pos[row], seq = a.seq ? a.seq[row] : row;
-  if (pos < 0) return;
-  if (pos >= a.t_max || seq < 0 || seq >= a.n_seqs) {
-    if (tid == 0) arcb_set_error(a.err, ARCB_DEV_BAD_INDEX);
-    return;
+  const float* p = a.proj + (size_t)row * a.pitch;
+  const int width = a.off_r + a.rotp;
+  float4 v[NV];
+  float sq = 0.f, sc = 0.f;
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int c = (tid + k * 128) * 4;
+    v[k] = c < width ? *reinterpret_cast<const float4*>(p + c) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
-  auto at = [&](int c) { return (((size_t)seq * ((a.kv_rankp + a.rotp) >> 6) + (c >> 6)) * a.t_max + pos) * 64 + (c & 63); };
-  for (int i = tid * 4; i < a.kv_rankp; i += STEP) st_act4(a.cache, at(i), normed(p + a.off_c, a.kv_norm, i, ic), a.fmt);
-  for (int i = tid * 4; i < a.rotp; i += STEP) {
-    const float4 v = *reinterpret_cast<const float4*>(p + a.off_r + i);
-    float4 o = v;
-    const int q = i >> 1;
-    if (q < a.pairs) {
-      const float2 c = __ldg(a.rot + (size_t)pos * a.pairs + q);
-      o.x = v.x * c.x - v.y * c.y;
-      o.y = v.y * c.x + v.x * c.y;
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int c = (tid + k * 128) * 4;
+    if (c < a.off_c) sq += sum_sq(v[k]);
+    else if (c < a.off_r) sc += sum_sq(v[k]);
+  }
+  sq = warp_sum(sq);
+  sc = warp_sum(sc);
+  if ((tid & 31) == 0) sm[tid >> 5] = make_float2(sq, sc);
+  __syncthreads();
+  sq = (sm[0].x + sm[1].x) + (sm[2].x + sm[3].x);
+  sc = (sm[0].y + sm[1].y) + (sm[2].y + sm[3].y);
+  const float iq = 1.f / sqrtf(sq / (float)a.q_rank + a.eps), ic = 1.f / sqrtf(sc / (float)a.kv_rank + a.eps);
+  const bool bad = pos >= a.t_max || seq < 0 || seq >= a.n_seqs;
+  if (bad && pos >= 0 && tid == 0) arcb_set_error(a.err, ARCB_DEV_BAD_INDEX);
+  const bool store = pos >= 0 && !bad;
+  const size_t row0 = ((size_t)seq * ((a.kv_rankp + a.rotp) >> 6) * a.t_max + pos) * 64, panel = (size_t)a.t_max * 64;
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int c = (tid + k * 128) * 4;
+    if (c < a.off_c) {
+      const float4 g = __ldg(reinterpret_cast<const float4*>(a.q_norm + c));
+      st_act4(a.cq, (size_t)row * a.q_rankp + c,
+              make_float4((v[k].x * iq) * g.x, (v[k].y * iq) * g.y, (v[k].z * iq) * g.z, (v[k].w * iq) * g.w), a.fmt);
+    } else if (c < width && store) {
+      float4 o = v[k];
+      if (c < a.off_r) {
+        const float4 g = __ldg(reinterpret_cast<const float4*>(a.kv_norm + c - a.off_c));
+        o = make_float4((o.x * ic) * g.x, (o.y * ic) * g.y, (o.z * ic) * g.z, (o.w * ic) * g.w);
+      } else if (a.rot) {
+        o = rotate4(o, __ldg(reinterpret_cast<const float4*>(a.rot + (size_t)pos * (a.rotp >> 1) + ((c - a.off_r) >> 1))));
+      }
+      const int cc = c - a.off_c;
+      st_act4(a.cache, row0 + (size_t)(cc >> 6) * panel + (cc & 63), o, a.fmt);
     }
-    if (q + 1 < a.pairs) {
-      const float2 c = __ldg(a.rot + (size_t)pos * a.pairs + q + 1);
-      o.z = v.z * c.x - v.w * c.y;
-      o.w = v.w * c.x + v.z * c.y;
-    }
-    st_act4(a.cache, at(a.kv_rankp + i), o, a.fmt);
   }
 }
 
@@ -310,8 +330,8 @@ __global__ void rot_table_kernel(float2* table, int t_max, int pairs, int dims, 
   const long long n = (long long)t_max * pairs;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
     const int p = (int)(i / pairs), k = (int)(i - (long long)p * pairs);
-    double s, c;
-    sincos(p * pow(base, -2.0 * k / dims), &s, &c);
+    double s = 0., c = 1.;
+    if (2 * k < dims) sincos(p * pow(base, -2.0 * k / dims), &s, &c);
     table[i] = make_float2((float)c, (float)s);
   }
 }
@@ -632,17 +652,23 @@ int arcb_launch_sandwich_norm(const SandwichArgs& a, cudaStream_t stream) {
 
 int arcb_launch_latent_prep(const LatentPrepArgs& a, cudaStream_t stream) {
   if (a.rows <= 0) return 0;
-  if (a.q_rankp % 4 || a.kv_rankp % 64 || a.rotp % 64 || a.off_c % 4 || a.off_r % 4 || a.pitch % 4) return -1;
-  const cudaError_t e = arcb_launch(latent_prep_kernel<4>, dim3(a.rows), dim3(128), 0, stream, a);
+  if (a.q_rankp % 4 || a.kv_rankp % 64 || a.rotp % 64 || a.pitch % 4 || a.off_c != a.q_rankp || a.off_r != a.off_c + a.kv_rankp) return -1;
+  const int steps = (a.off_r + a.rotp + 511) / 512;
+  const dim3 grid(a.rows), block(128);
+  const cudaError_t e = steps <= 1   ? arcb_launch(latent_prep_kernel<1>, grid, block, 0, stream, a)
+                        : steps <= 3 ? arcb_launch(latent_prep_kernel<3>, grid, block, 0, stream, a)
+                        : steps <= 6 ? arcb_launch(latent_prep_kernel<6>, grid, block, 0, stream, a)
+                        : steps <= 12 ? arcb_launch(latent_prep_kernel<12>, grid, block, 0, stream, a)
+                                      : cudaErrorInvalidValue;
   arcb_count_launch(1);
   return (int)e;
 }
 
-int arcb_launch_rot_table(float2* table, int t_max, int dims, double base, cudaStream_t stream) {
-  if (t_max <= 0 || dims < 2) return 0;
-  long long blocks = ((long long)t_max * (dims / 2) + 255) / 256;
+int arcb_launch_rot_table(float2* table, int t_max, int pairs, int dims, double base, cudaStream_t stream) {
+  if (t_max <= 0 || pairs <= 0) return 0;
+  long long blocks = ((long long)t_max * pairs + 255) / 256;
   if (blocks > 148 * 8) blocks = 148 * 8;
-  rot_table_kernel<<<(unsigned)blocks, 256, 0, stream>>>(table, t_max, dims / 2, dims, base);
+  rot_table_kernel<<<(unsigned)blocks, 256, 0, stream>>>(table, t_max, pairs, dims, base);
   arcb_count_launch(1);
   return (int)cudaGetLastError();
 }

@@ -30,7 +30,9 @@ struct LmEmbedArgs {
   const float* embed;      // [vocab][pitch]
   float alpha;             // x leaves multiplied by the residual factor of the first sublayer
   float* x;                // [rows][pitch]
-  void* xn;                // [rows][pitch] activation format
+  void* xn;                // [rows][pitch] activation format, null: not written
+  int* zero;               // optional counters the pass starts from
+  int n_zero;
 };
 
 // y = norm(x) * w; xn gets y in the activation format, and x (optional) y * x_scale.
@@ -72,8 +74,7 @@ struct LatentPrepArgs {
   const float* q_norm;     // [q_rankp]
   const float* kv_norm;    // [kv_rankp]
   float eps;
-  const float2* rot;       // [t_max][pairs] (cos, sin)
-  int pairs;
+  const float2* rot;       // [t_max][rotp / 2] (cos, sin), null: nothing turns
   void* cq;                // [rows][q_rankp]
   void* cache;             // [n_seqs][(kv_rankp + rotp) / 64][t_max][64]
   const int* pos;          // [rows], negative: the row stores nothing
@@ -98,8 +99,8 @@ int arcb_launch_step_begin(const StepState& st, const LmEmbedArgs& a, cudaStream
 int arcb_launch_lm_norm(const LmNormArgs& a, cudaStream_t stream);
 int arcb_launch_sandwich_norm(const SandwichArgs& a, cudaStream_t stream);
 int arcb_launch_latent_prep(const LatentPrepArgs& a, cudaStream_t stream);
-// table[p][i] = (cos, sin)(p * base^(-2 i / dims)), i < dims / 2
-int arcb_launch_rot_table(float2* table, int t_max, int dims, double base, cudaStream_t stream);
+// table[p][i] = (cos, sin)(p * base^(-2 i / dims)), i < dims / 2, and (1, 0) for i from there to pairs - 1
+int arcb_launch_rot_table(float2* table, int t_max, int pairs, int dims, double base, cudaStream_t stream);
 int arcb_launch_proj_prep(const ProjArgs& a, const float* proj, cudaStream_t stream);
 int arcb_launch_pick(const PickArgs& a, const StepState& st, cudaStream_t stream);
 int arcb_launch_seg_commit(const StepState& st, const int* seg_seq, const int* seg_pos0, const int* seg_rows, int n,

@@ -1,31 +1,17 @@
 // Routing of tokens to experts, on the device without a host round trip:
 //   route   : sigmoid of the router logits (fp32), the `top` largest scores of every row (the first of equal ones),
 //             and the row's place among the tokens of each chosen expert
-//   plan    : slots of every expert (padded to whole tiles of the grouped product), expert of every tile
-//   scatter : rows of xn in slot order, slot and weight of every (row, choice)
+//   scatter : slots of every expert (padded to whole tiles of the grouped product), expert of every tile, rows of xn
+//             in slot order, slot and weight of every (row, choice)
 // Slots of one expert are filled in no particular order: a row's result does not depend on its slot.
 #include "launch.cuh"
 #include "moe.cuh"
 
 namespace {
 
-constexpr int PER_LANE = MOE_MAX_EXPERTS / 32;
-constexpr int PLAN_THREADS = 256;
-static_assert(PLAN_THREADS == MOE_MAX_EXPERTS, "one thread of the plan per expert");
-
-// One warp per row; lane i holds the scores of experts i, i + 32, ...
-__global__ void __launch_bounds__(128)
-moe_route_kernel(MoeArgs a) {
-  pdl_launch_dependents();
-  pdl_wait();
-  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (row >= a.rows) return;
-  float s[PER_LANE];
-#pragma unroll
-  for (int i = 0; i < PER_LANE; ++i) {
-    const int e = lane + 32 * i;
-    s[i] = e < a.experts ? 1.f / (1.f + expf(-a.z[(size_t)row * a.z_pitch + e])) : -1.f;
-  }
+// The chosen experts of a row by one warp; lane i holds the scores of experts i, i + 32, ... in s.
+template <int PER_LANE>
+__device__ __forceinline__ void choose(const MoeArgs& a, int row, int lane, float (&s)[PER_LANE]) {
   int my_e = 0;
   float my_w = 0.f;
   for (int k = 0; k < a.top; ++k) {
@@ -33,9 +19,8 @@ moe_route_kernel(MoeArgs a) {
     unsigned long long best = 0;
 #pragma unroll
     for (int i = 0; i < PER_LANE; ++i) {
-      const int e = lane + 32 * i;
       if (s[i] >= 0.f) {
-        const unsigned long long key = ((unsigned long long)(__float_as_uint(s[i]) + 1u) << 32) | (uint32_t)~e;
+        const unsigned long long key = ((unsigned long long)(__float_as_uint(s[i]) + 1u) << 32) | (uint32_t)~(lane + 32 * i);
         best = key > best ? key : best;
       }
     }
@@ -61,52 +46,128 @@ moe_route_kernel(MoeArgs a) {
   }
 }
 
-// One CTA, one thread per expert.
-__global__ void __launch_bounds__(PLAN_THREADS)
-moe_plan_kernel(MoeArgs a) {
+__device__ __forceinline__ float score(float z) { return 1.f / (1.f + expf(-z)); }
+
+// One warp per row.
+template <int PER_LANE>
+__global__ void __launch_bounds__(128)
+moe_route_kernel(MoeArgs a) {
   pdl_launch_dependents();
   pdl_wait();
-  __shared__ int scan[PLAN_THREADS];
-  const int e = threadIdx.x;
-  const int n = e < a.experts ? a.count[e] : 0;
-  const int padded = (n + a.gran - 1) / a.gran * a.gran;
-  scan[e] = padded;
-  __syncthreads();
+  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= a.rows) return;
+  float s[PER_LANE];
 #pragma unroll
-  for (int o = 1; o < PLAN_THREADS; o <<= 1) {
-    const int v = e >= o ? scan[e - o] : 0;
-    __syncthreads();
-    scan[e] += v;
-    __syncthreads();
+  for (int i = 0; i < PER_LANE; ++i) {
+    const int e = lane + 32 * i;
+    s[i] = e < a.experts ? score(a.z[(size_t)row * a.z_pitch + e]) : -1.f;
   }
-  const int first = scan[e] - padded;
-  if (e < a.experts) {
-    a.offset[e] = first;
-    a.count[e] = 0;
-    for (int t = 0; t < padded; t += 128) a.tile_expert[(first + t) >> 7] = e;
-    for (int i = n; i < padded; ++i) a.slot_weight[first + i] = 0.f;
-  }
-  if (e == PLAN_THREADS - 1) *a.n_tiles = scan[e] >> 7;
+  choose<PER_LANE>(a, row, lane, s);
 }
 
-// One warp per (row, choice).
-__global__ void __launch_bounds__(128)
+// One CTA of eight warps per row, which also multiplies the row with the router (16-bit formats).
+constexpr int ROUTER_WARPS = 8;
+__global__ void __launch_bounds__(ROUTER_WARPS * 32)
+moe_router_kernel(MoeArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float s_z[MOE_MAX_EXPERTS];
+  const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const uint4* x = reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(a.xn) + (size_t)row * a.pitch);
+  const int n = a.pitch / 8;                             // 8 columns a load
+  for (int e0 = warp * 4; e0 < a.experts; e0 += ROUTER_WARPS * 4) {
+    float d[4] = {0.f, 0.f, 0.f, 0.f};
+    const uint4* w = reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(a.w_router) + (size_t)e0 * a.pitch);
+    for (int i = lane; i < n; i += 32) {                 // rows behind the last expert are zero
+      const uint4 xv = x[i];
+      const uint32_t xr[4] = {xv.x, xv.y, xv.z, xv.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const uint4 wv = __ldg(w + (size_t)e * n + i);
+        const uint32_t wr[4] = {wv.x, wv.y, wv.z, wv.w};
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float2 p = unpack2_act(xr[j], a.fmt), q = unpack2_act(wr[j], a.fmt);
+          d[e] = fmaf(p.x, q.x, d[e]);
+          d[e] = fmaf(p.y, q.y, d[e]);
+        }
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      d[e] = warp_sum(d[e]);
+      if (lane == 0 && e0 + e < a.experts) s_z[e0 + e] = d[e];
+    }
+  }
+  __syncthreads();
+  if (warp) return;
+  float s[MOE_MAX_EXPERTS / 32];
+#pragma unroll
+  for (int i = 0; i < MOE_MAX_EXPERTS / 32; ++i) {
+    const int e = lane + 32 * i;
+    s[i] = e < a.experts ? score(s_z[e]) : -1.f;
+  }
+  choose<MOE_MAX_EXPERTS / 32>(a, row, lane, s);
+}
+
+// One CTA per row.  Every CTA takes the running sum over the experts' padded counts for itself; the first one also
+// lists the tiles and clears the padding slots' weights.
+constexpr int SCATTER_THREADS = 128;
+__global__ void __launch_bounds__(SCATTER_THREADS)
 moe_scatter_kernel(MoeArgs a) {
   pdl_launch_dependents();
   pdl_wait();
-  const long long w = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
-  const int lane = threadIdx.x & 31;
-  if (w >= (long long)a.rows * a.top) return;
-  const int row = (int)(w / a.top);
-  const int slot = a.offset[a.expert[w]] + a.rank[w];
-  if (lane == 0) {
-    a.slot[w] = slot;
-    a.slot_weight[slot] = a.weight[w];
+  __shared__ int s_first[MOE_MAX_EXPERTS + 1];
+  __shared__ int s_slot[MOE_MAX_TOP];
+  __shared__ int s_warp[2 * SCATTER_THREADS / 32];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  int incl[2], padded[2];                                // experts tid and tid + 128
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int e = tid + i * SCATTER_THREADS;
+    padded[i] = e < a.experts ? (a.count[e] + a.gran - 1) / a.gran * a.gran : 0;
+    int v = padded[i];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int t = __shfl_up_sync(0xffffffffu, v, o);
+      if (lane >= o) v += t;
+    }
+    incl[i] = v;
+    if (lane == 31) s_warp[i * (SCATTER_THREADS / 32) + warp] = v;
   }
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    int before = 0;
+    for (int j = 0; j < i * (SCATTER_THREADS / 32) + warp; ++j) before += s_warp[j];
+    const int e = tid + i * SCATTER_THREADS;
+    s_first[e] = before + incl[i] - padded[i];
+    if (e == MOE_MAX_EXPERTS - 1) s_first[MOE_MAX_EXPERTS] = before + incl[i];
+  }
+  __syncthreads();
+  const int row = blockIdx.x;
+  if (row == 0) {
+    for (int e = warp; e < a.experts; e += SCATTER_THREADS / 32) {
+      const int first = s_first[e], n = a.count[e], end = (n + a.gran - 1) / a.gran * a.gran;
+      for (int t = lane * 128; t < end; t += 32 * 128) a.tile_expert[(first + t) >> 7] = e;
+      for (int i = n + lane; i < end; i += 32) a.slot_weight[first + i] = 0.f;
+    }
+    if (tid == 0) *a.n_tiles = s_first[MOE_MAX_EXPERTS] >> 7;
+  }
+  if (tid < a.top) {
+    const size_t at = (size_t)row * a.top + tid;
+    const int slot = s_first[a.expert[at]] + a.rank[at];
+    s_slot[tid] = slot;
+    a.slot[at] = slot;
+    a.slot_weight[slot] = a.weight[at];
+  }
+  __syncthreads();
   const size_t bytes = (size_t)a.pitch * act_bytes(a.fmt);
   const uint4* src = reinterpret_cast<const uint4*>(reinterpret_cast<const uint8_t*>(a.xn) + row * bytes);
-  uint4* dst = reinterpret_cast<uint4*>(reinterpret_cast<uint8_t*>(a.xs) + slot * bytes);
-  for (int i = lane; i < (int)(bytes / 16); i += 32) dst[i] = src[i];
+  for (int i = tid; i < (int)(bytes / 16); i += SCATTER_THREADS) {
+    const uint4 v = src[i];
+    for (int k = 0; k < a.top; ++k) reinterpret_cast<uint4*>(reinterpret_cast<uint8_t*>(a.xs) + s_slot[k] * bytes)[i] = v;
+  }
 }
 
 }  // namespace
@@ -118,16 +179,22 @@ int arcb_moe_max_slots(int rows, int experts, int top, int gran) {
   return (int)((s + gran - 1) / gran * gran);
 }
 
+bool arcb_moe_router_inside(int rows, int experts, int pitch, int fmt) {
+  return fmt != 2 && (long long)rows * experts * pitch <= 32ll << 20;     // 64 MB of weights through the L2 cache
+}
+
 int arcb_launch_moe_route(const MoeArgs& a, cudaStream_t stream) {
   if (a.rows <= 0) return 0;
-  if (a.experts > MOE_MAX_EXPERTS || a.top > MOE_MAX_TOP || a.top > a.experts || a.top < 1) return -1;
+  if (a.experts > MOE_MAX_EXPERTS || a.top > MOE_MAX_TOP || a.top > a.experts || a.top < 1 || a.pitch % 8) return -1;
   if (a.max_slots < arcb_moe_max_slots(a.rows, a.experts, a.top, a.gran)) return -1;
-  cudaError_t e = arcb_launch(moe_route_kernel, dim3((a.rows + 3) / 4), dim3(128), 0, stream, a);
+  const dim3 rows4((a.rows + 3) / 4);
+  cudaError_t e = !a.z ? arcb_launch(moe_router_kernel, dim3(a.rows), dim3(ROUTER_WARPS * 32), 0, stream, a)
+                  : a.experts <= 32  ? arcb_launch(moe_route_kernel<1>, rows4, dim3(128), 0, stream, a)
+                  : a.experts <= 64  ? arcb_launch(moe_route_kernel<2>, rows4, dim3(128), 0, stream, a)
+                  : a.experts <= 128 ? arcb_launch(moe_route_kernel<4>, rows4, dim3(128), 0, stream, a)
+                                     : arcb_launch(moe_route_kernel<8>, rows4, dim3(128), 0, stream, a);
   if (e != cudaSuccess) return (int)e;
-  e = arcb_launch(moe_plan_kernel, dim3(1), dim3(PLAN_THREADS), 0, stream, a);
-  if (e != cudaSuccess) return (int)e;
-  const long long n = ((long long)a.rows * a.top + 3) / 4;
-  e = arcb_launch(moe_scatter_kernel, dim3((unsigned)n), dim3(128), 0, stream, a);
-  arcb_count_launch(3);
+  e = arcb_launch(moe_scatter_kernel, dim3(a.rows), dim3(SCATTER_THREADS), 0, stream, a);
+  arcb_count_launch(2);
   return (int)e;
 }
