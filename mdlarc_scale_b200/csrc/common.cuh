@@ -58,6 +58,19 @@ __device__ __forceinline__ uint32_t pack2_act_chk(float a, float b, int act_f16,
   return pack2_act(a, b, act_f16);
 }
 
+// pack2_act in one conversion (which clamps to the finite range); `amax` collects the largest magnitude for a
+// saturation check by the caller
+__device__ __forceinline__ uint32_t pack2_act_max(float a, float b, int act_f16, float& amax) {
+  if (act_f16) {
+    uint32_t d;
+    asm("cvt.rn.satfinite.f16x2.f32 %0, %1, %2;" : "=r"(d) : "f"(b), "f"(a));
+    amax = fmaxf(fmaxf(amax, fabsf(a)), fabsf(b));
+    return d;
+  }
+  __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  return *reinterpret_cast<uint32_t*>(&h);
+}
+
 __device__ __forceinline__ float2 unpack2_act(uint32_t v, int act_f16) {
   if (act_f16) {
     __half2 h = *reinterpret_cast<__half2*>(&v);

@@ -25,9 +25,9 @@ constexpr int TC_BK = 64;  // 64 x 2 B = one 128-byte swizzle row
 constexpr int TC_EPI_WARPS = 8;                  // two warps per TMEM lane quarter, half of the columns each
 constexpr int TC_THREADS = 64 + 32 * TC_EPI_WARPS;
 
-template <int BN>
+template <int BN, int MODE = EPI_STORE_F32>
 struct TcCfg {
-  static constexpr int STAGES = (BN == 256) ? 4 : 6;
+  static constexpr int STAGES = (BN == 256) ? (MODE == EPI_ACT ? 3 : 4) : MODE == EPI_ACT ? 5 : 6;
   static constexpr int A_BYTES = TC_BM * TC_BK * 2;
   static constexpr int B_BYTES = BN * TC_BK * 2;
   static constexpr int STAGE_BYTES = A_BYTES + B_BYTES;
@@ -39,10 +39,13 @@ struct TcCfg {
 // The residual epilogue stages 128 x 32 fp32 chunks in shared memory (one 16 KB buffer per group of
 // four epilogue warps) and adds them to the residual stream with a bulk tensor reduce.
 constexpr int EPI_STAGE_GROUP_BYTES = 128 * 32 * 4;
+// EPI_ACT products may be short (a few K blocks a tile), so its boxes leave through two buffers in turn
+template <int MODE>
+__host__ __device__ constexpr int epi_group_bytes() { return (MODE == EPI_ACT ? 2 : 1) * EPI_STAGE_GROUP_BYTES; }
 template <int MODE>
 __host__ __device__ constexpr int epi_stage_bytes() {
-  return (MODE == EPI_RESID || MODE == EPI_SWIGLU || MODE == EPI_QKV_ROPE || MODE == EPI_RELU2 ||
-          MODE == EPI_HEADS || MODE == EPI_ACT || MODE == EPI_GLU) ? 2 * EPI_STAGE_GROUP_BYTES : 0;
+  return MODE == EPI_ACT ? 2 * epi_group_bytes<MODE>() : (MODE == EPI_RESID || MODE == EPI_SWIGLU || MODE == EPI_QKV_ROPE || MODE == EPI_RELU2 ||
+          MODE == EPI_HEADS || MODE == EPI_GLU) ? 2 * EPI_STAGE_GROUP_BYTES : 0;
 }
 // epilogues that go through the staging buffers and the third tensor map
 template <int BN, int MODE>
@@ -200,17 +203,18 @@ __device__ __forceinline__ void epilogue_relu2_tma(const GemmEpilogue& ep, const
 template <int BN>
 __device__ __forceinline__ void epilogue_act_tma(const GemmEpilogue& ep, const CUtensorMap* tmap_h, uint32_t t_row, int m0,
                                                  bool row_ok, int n_tile0, int grp, int row_in_tile, uint32_t stage_smem,
-                                                 uint8_t* stage_ptr, bool elected) {
-  uint8_t* my_row = stage_ptr + row_in_tile * 128;
+                                                 uint8_t* stage_ptr, uint32_t& turn, bool elected) {
   const int sw = row_in_tile & 7;
+  float amax = 0.f;
   const float2* cs = (ep.rot.table && row_ok) ? rot_row(ep, m0 + row_in_tile) : nullptr;
 #pragma unroll 1
   for (int b = grp * (BN / 128); b < (grp + 1) * (BN / 128); ++b) {
     const int n0 = n_tile0 + b * 64;
     if (n0 >= ep.N) break;               // uniform over the group
     const int in_rot = cs ? n0 % ep.rot.head - ep.rot.off : -1;
-    if (elected) bulk_wait_read_all();   // the previous store has read the buffer
+    if (elected) bulk_wait_read_but_one();   // the store before the previous one has read this buffer
     named_bar_sync(1 + grp, 128);
+    uint8_t* my_row = stage_ptr + turn * EPI_STAGE_GROUP_BYTES + row_in_tile * 128;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
       uint32_t r[32];
@@ -238,17 +242,19 @@ __device__ __forceinline__ void epilogue_act_tma(const GemmEpilogue& ep, const C
         uint32_t w[4];
 #pragma unroll
         for (int i = 0; i < 4; ++i)
-          w[i] = pack2_act_chk(__uint_as_float(r[8 * q + 2 * i]), __uint_as_float(r[8 * q + 2 * i + 1]), ep.act_f16, ep.err);
+          w[i] = pack2_act_max(__uint_as_float(r[8 * q + 2 * i]), __uint_as_float(r[8 * q + 2 * i + 1]), ep.act_f16, amax);
         *reinterpret_cast<uint4*>(my_row + (((half * 4 + q) ^ sw) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
       }
     }
     fence_proxy_async_smem();
     named_bar_sync(1 + grp, 128);
-    if (elected && m0 < ep.M) {
-      tma_store_2d(tmap_h, stage_smem, n0, m0);
+    if (elected) {
+      if (m0 < ep.M) tma_store_2d(tmap_h, stage_smem + turn * EPI_STAGE_GROUP_BYTES, n0, m0);
       bulk_commit_group();
     }
+    turn ^= 1;
   }
+  if (amax > 65504.f && row_ok) arcb_count_saturation(ep.err);
 }
 
 // Fused mixer projection (ProjArgs), this group's column half of the tile, 64 columns at a time.  A 64-column
@@ -560,7 +566,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
                const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ CUtensorMap tmap_y,
                const __grid_constant__ CUtensorMap tmap_z, GemmEpilogue ep, int K, uint32_t idesc, int tiles_n,
                int tiles_total) {
-  using Cfg = TcCfg<BN>;
+  using Cfg = TcCfg<BN, MODE>;
   pdl_launch_dependents();
   extern __shared__ uint8_t smem_raw[];
   const uint32_t raw = smem_u32(smem_raw);
@@ -678,6 +684,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
     const int quarter = warp & 3;
     const int col_half = (warp - 2) >> 2;
     const int row_in_tile = quarter * 32 + lane;
+    [[maybe_unused]] uint32_t turn = 0;
     uint32_t it = 0;
     for (int tile = blockIdx.x; tile < tiles_total; tile += gridDim.x, ++it) {
       const int m_blk = tile / tiles_n, n_blk = tile - m_blk * tiles_n;
@@ -706,8 +713,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
                                base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
       else if constexpr (MODE == EPI_ACT && BN >= 128)
         epilogue_act_tma<BN>(ep, &tmap_x, t_row, m_blk * TC_BM, row_ok, n_blk * BN, col_half, row_in_tile,
-                             base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
-                             base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
+                             base + RING_BYTES + col_half * epi_group_bytes<MODE>(),
+                             base_ptr + RING_BYTES + col_half * epi_group_bytes<MODE>(), turn, quarter == 0 && lane == 0);
       else if constexpr ((MODE == EPI_SWIGLU || MODE == EPI_GLU) && BN == 256)
         epilogue_swiglu_tma<MODE>(ep, &tmap_x, t_row + col_half * 128, m_blk * TC_BM, n_blk * BN + col_half * 128, col_half,
                             row_in_tile, base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
@@ -753,7 +760,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
 template <int MODE>
 struct Tc2Cfg {
   static constexpr int BN = 256;
-  static constexpr int STAGES = (MODE == EPI_QKV_ROPE) ? 5 : 6;
+  static constexpr int STAGES = (MODE == EPI_QKV_ROPE || MODE == EPI_ACT) ? 5 : 6;
   static constexpr int A_BYTES = TC_BM * TC_BK * 2;   // this CTA's 128 rows of A
   static constexpr int B_BYTES = 128 * TC_BK * 2;     // this CTA's 128 rows of W
   static constexpr int STAGE_BYTES = A_BYTES + B_BYTES;
@@ -892,6 +899,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constan
     const int quarter = warp & 3;
     const int col_half = (warp - 2) >> 2;
     const int row_in_tile = quarter * 32 + lane;
+    [[maybe_unused]] uint32_t turn = 0;
     uint32_t it = 0;
     for (int tile = pair; tile < tiles_total; tile += n_pairs, ++it) {
       const int m_blk = tile / tiles_n, n_blk = tile - m_blk * tiles_n;
@@ -919,8 +927,8 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constan
                                base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
       else if constexpr (MODE == EPI_ACT)
         epilogue_act_tma<BN>(ep, &tmap_x, t_row, m_blk * 256 + (int)rank * 128, row_ok, n_blk * BN, col_half, row_in_tile,
-                             base + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES,
-                             base_ptr + RING_BYTES + col_half * EPI_STAGE_GROUP_BYTES, quarter == 0 && lane == 0);
+                             base + RING_BYTES + col_half * epi_group_bytes<MODE>(),
+                             base_ptr + RING_BYTES + col_half * epi_group_bytes<MODE>(), turn, quarter == 0 && lane == 0);
       else if constexpr (MODE == EPI_SWIGLU || MODE == EPI_GLU)
         epilogue_swiglu_tma<MODE>(ep, &tmap_x, t_row + col_half * 128, m_blk * 256 + (int)rank * 128,
                             n_blk * BN + col_half * 128, col_half, row_in_tile,
@@ -1367,10 +1375,10 @@ bool arcb_gemm_tc_supported(int M, int N, int K) {
 template <int MODE>
 static cudaError_t set_tc_smem_attr() {
   cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<128, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                       TcCfg<128>::SMEM_BYTES + epi_stage_bytes<MODE>());
+                                       TcCfg<128, MODE>::SMEM_BYTES + epi_stage_bytes<MODE>());
   if (e != cudaSuccess) return e;
   return cudaFuncSetAttribute(gemm_tc_kernel<256, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                              TcCfg<256>::SMEM_BYTES + epi_stage_bytes<MODE>());
+                              TcCfg<256, MODE>::SMEM_BYTES + epi_stage_bytes<MODE>());
 }
 
 // Per-device launch limits, filled by arcb_gemm_init() for the device that is current then and
@@ -1405,7 +1413,7 @@ int arcb_gemm_init() {
   if ((e = set_tc_smem_attr<EPI_HEADS>()) != cudaSuccess) return (int)e;
   if ((e = set_tc_smem_attr<EPI_ACT>()) != cudaSuccess) return (int)e;
   if ((e = cudaFuncSetAttribute(gemm_tc_kernel<64, EPI_ACT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                TcCfg<64>::SMEM_BYTES + epi_stage_bytes<EPI_ACT>())) != cudaSuccess) return (int)e;
+                                TcCfg<64, EPI_ACT>::SMEM_BYTES + epi_stage_bytes<EPI_ACT>())) != cudaSuccess) return (int)e;
   if ((e = set_tc_smem_attr<EPI_GLU>()) != cudaSuccess) return (int)e;
   if ((e = set_tc2_smem_attr<EPI_ACT>()) != cudaSuccess) return (int)e;
   if ((e = set_tc2_smem_attr<EPI_GLU>()) != cudaSuccess) return (int)e;
@@ -1450,7 +1458,7 @@ static cudaError_t launch_tc(const CUtensorMap& ta, const CUtensorMap& tb, const
   const int sms = num_sms();
   const uint32_t idesc = umma_idesc_f16(TC_BM, BN, act_f16 ? 0 : 1, act_f16 ? 0 : 1);
   return arcb_launch(gemm_tc_kernel<BN, MODE>, dim3(tiles < sms ? tiles : sms), dim3(TC_THREADS),
-                     TcCfg<BN>::SMEM_BYTES + epi_stage_bytes<MODE>(), stream, ta, tb, tx, ty, tz, ep, K, idesc, tiles_n,
+                     TcCfg<BN, MODE>::SMEM_BYTES + epi_stage_bytes<MODE>(), stream, ta, tb, tx, ty, tz, ep, K, idesc, tiles_n,
                      tiles);
 }
 

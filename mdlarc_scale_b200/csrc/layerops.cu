@@ -174,8 +174,9 @@ __device__ __forceinline__ float cta_sum(float v, float* sm) {
 
 __device__ __forceinline__ float sum_sq(float4 v) { return (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w); }
 
-// One CTA of four warps per row; NV float4 per thread hold the row (REGS) or every pass reads it again.
-template <int NV, bool REGS>
+// One CTA of four warps per row; NV float4 per thread hold the row (REGS) or every pass reads it again.  AHEAD: the
+// residual row is loaded beside the sublayer's output (few rows: shorter; many rows: the registers are worth more).
+template <int NV, bool REGS, bool AHEAD>
 __global__ void __launch_bounds__(128)
 sandwich_norm_kernel(SandwichArgs a) {
   pdl_launch_dependents();
@@ -219,15 +220,15 @@ sandwich_norm_kernel(SandwichArgs a) {
   };
   // padding columns are zero in y, x, the embedding and the gains
   if constexpr (REGS) {
-    float4 v[NV], r[NV];
+    float4 v[NV], r[AHEAD ? NV : 1];
     float ss = 0.f;
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
       const int i = (tid + k * 128) * 4;
-      v[k] = r[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+      v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (i < a.pitch) {
+        if constexpr (AHEAD) r[k] = *reinterpret_cast<const float4*>(x + i);
         v[k] = sublayer(i);
-        r[k] = *reinterpret_cast<const float4*>(x + i);
       }
       ss += sum_sq(v[k]);
     }
@@ -237,7 +238,7 @@ sandwich_norm_kernel(SandwichArgs a) {
     for (int k = 0; k < NV; ++k) {
       const int i = (tid + k * 128) * 4;
       if (i >= a.pitch) continue;
-      v[k] = added(i, r[k], v[k], inv);
+      v[k] = added(i, AHEAD ? r[AHEAD ? k : 0] : *reinterpret_cast<const float4*>(x + i), v[k], inv);
       if (a.dense) dense(i, v[k]);
       v[k] = with_embed(i, v[k]);
       *reinterpret_cast<float4*>(x + i) = v[k];
@@ -642,10 +643,14 @@ int arcb_launch_sandwich_norm(const SandwichArgs& a, cudaStream_t stream) {
   if (a.rows <= 0) return 0;
   if (a.pitch % 128) return -1;
   const dim3 grid(a.rows), block(128);
-  const cudaError_t e = a.pitch <= 512 * 2   ? arcb_launch(sandwich_norm_kernel<2, true>, grid, block, 0, stream, a)
-                        : a.pitch <= 512 * 4 ? arcb_launch(sandwich_norm_kernel<4, true>, grid, block, 0, stream, a)
-                        : a.pitch <= 512 * 8 ? arcb_launch(sandwich_norm_kernel<8, true>, grid, block, 0, stream, a)
-                                             : arcb_launch(sandwich_norm_kernel<1, false>, grid, block, 0, stream, a);
+  const int steps = (a.pitch + 511) / 512;
+  const bool ahead = a.rows <= 1024;
+  auto go = [&](auto few, auto many) { return arcb_launch(ahead ? few : many, grid, block, 0, stream, a); };
+  const cudaError_t e = steps <= 2   ? go(sandwich_norm_kernel<2, true, true>, sandwich_norm_kernel<2, true, false>)
+                        : steps <= 3 ? go(sandwich_norm_kernel<3, true, true>, sandwich_norm_kernel<3, true, false>)
+                        : steps <= 4 ? go(sandwich_norm_kernel<4, true, true>, sandwich_norm_kernel<4, true, false>)
+                        : steps <= 8 ? go(sandwich_norm_kernel<8, true, true>, sandwich_norm_kernel<8, true, false>)
+                                     : arcb_launch(sandwich_norm_kernel<1, false, false>, grid, block, 0, stream, a);
   arcb_count_launch(1);
   return (int)e;
 }

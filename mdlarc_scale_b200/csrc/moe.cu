@@ -9,11 +9,12 @@
 
 namespace {
 
-// The chosen experts of a row by one warp; lane i holds the scores of experts i, i + 32, ... in s.
+// The chosen experts of a row by one warp; lane i holds the scores of experts i, i + 32, ... in s.  Lane k returns
+// the k-th choice.
 template <int PER_LANE>
-__device__ __forceinline__ void choose(const MoeArgs& a, int row, int lane, float (&s)[PER_LANE]) {
+__device__ __forceinline__ int choose(const MoeArgs& a, int lane, float (&s)[PER_LANE], float& my_w) {
   int my_e = 0;
-  float my_w = 0.f;
+  my_w = 0.f;
   for (int k = 0; k < a.top; ++k) {
     // scores lie in [0, 1]: their bits order like the numbers, and ~e prefers the first of equal ones
     unsigned long long best = 0;
@@ -38,35 +39,55 @@ __device__ __forceinline__ void choose(const MoeArgs& a, int row, int lane, floa
     for (int i = 0; i < PER_LANE; ++i)
       if (lane + 32 * i == e) s[i] = -1.f;
   }
-  if (lane < a.top) {
-    const size_t at = (size_t)row * a.top + lane;
-    a.expert[at] = my_e;
-    a.weight[at] = my_w;
-    a.rank[at] = atomicAdd(a.count + my_e, 1);
-  }
+  return my_e;
 }
 
 __device__ __forceinline__ float score(float z) { return 1.f / (1.f + expf(-z)); }
 
-// One warp per row.
+// One warp per row and turn; ranks are counted within the CTA first, so that an expert's counter is touched once per CTA.
+constexpr int ROUTE_ROWS = 32;
 template <int PER_LANE>
 __global__ void __launch_bounds__(128)
 moe_route_kernel(MoeArgs a) {
   pdl_launch_dependents();
   pdl_wait();
-  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (row >= a.rows) return;
-  float s[PER_LANE];
+  __shared__ int s_count[MOE_MAX_EXPERTS], s_base[MOE_MAX_EXPERTS];
+  const int row0 = blockIdx.x * ROUTE_ROWS, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int e = threadIdx.x; e < a.experts; e += 128) s_count[e] = 0;
+  __syncthreads();
+  int my_e[ROUTE_ROWS / 4], my_r[ROUTE_ROWS / 4];
 #pragma unroll
-  for (int i = 0; i < PER_LANE; ++i) {
-    const int e = lane + 32 * i;
-    s[i] = e < a.experts ? score(a.z[(size_t)row * a.z_pitch + e]) : -1.f;
+  for (int t = 0; t < ROUTE_ROWS / 4; ++t) {
+    const int row = row0 + t * 4 + warp;
+    my_e[t] = my_r[t] = 0;
+    if (row >= a.rows) continue;
+    float s[PER_LANE];
+#pragma unroll
+    for (int i = 0; i < PER_LANE; ++i) {
+      const int e = lane + 32 * i;
+      s[i] = e < a.experts ? score(a.z[(size_t)row * a.z_pitch + e]) : -1.f;
+    }
+    float w;
+    my_e[t] = choose<PER_LANE>(a, lane, s, w);
+    if (lane < a.top) {
+      a.expert[(size_t)row * a.top + lane] = my_e[t];
+      a.weight[(size_t)row * a.top + lane] = w;
+      my_r[t] = atomicAdd(s_count + my_e[t], 1);
+    }
   }
-  choose<PER_LANE>(a, row, lane, s);
+  __syncthreads();
+  for (int e = threadIdx.x; e < a.experts; e += 128) s_base[e] = s_count[e] ? atomicAdd(a.count + e, s_count[e]) : 0;
+  __syncthreads();
+#pragma unroll
+  for (int t = 0; t < ROUTE_ROWS / 4; ++t) {
+    const int row = row0 + t * 4 + warp;
+    if (row < a.rows && lane < a.top) a.rank[(size_t)row * a.top + lane] = s_base[my_e[t]] + my_r[t];
+  }
 }
 
 // One CTA of eight warps per row, which also multiplies the row with the router (16-bit formats).
 constexpr int ROUTER_WARPS = 8;
+template <int PER_LANE>
 __global__ void __launch_bounds__(ROUTER_WARPS * 32)
 moe_router_kernel(MoeArgs a) {
   pdl_launch_dependents();
@@ -78,6 +99,7 @@ moe_router_kernel(MoeArgs a) {
   for (int e0 = warp * 4; e0 < a.experts; e0 += ROUTER_WARPS * 4) {
     float d[4] = {0.f, 0.f, 0.f, 0.f};
     const uint4* w = reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(a.w_router) + (size_t)e0 * a.pitch);
+#pragma unroll 4
     for (int i = lane; i < n; i += 32) {                 // rows behind the last expert are zero
       const uint4 xv = x[i];
       const uint32_t xr[4] = {xv.x, xv.y, xv.z, xv.w};
@@ -101,13 +123,20 @@ moe_router_kernel(MoeArgs a) {
   }
   __syncthreads();
   if (warp) return;
-  float s[MOE_MAX_EXPERTS / 32];
+  float s[PER_LANE];
 #pragma unroll
-  for (int i = 0; i < MOE_MAX_EXPERTS / 32; ++i) {
+  for (int i = 0; i < PER_LANE; ++i) {
     const int e = lane + 32 * i;
     s[i] = e < a.experts ? score(s_z[e]) : -1.f;
   }
-  choose<MOE_MAX_EXPERTS / 32>(a, row, lane, s);
+  float w;
+  const int e = choose<PER_LANE>(a, lane, s, w);
+  if (lane < a.top) {
+    const size_t at = (size_t)row * a.top + lane;
+    a.expert[at] = e;
+    a.weight[at] = w;
+    a.rank[at] = atomicAdd(a.count + e, 1);
+  }
 }
 
 // One CTA per row.  Every CTA takes the running sum over the experts' padded counts for itself; the first one also
@@ -187,12 +216,14 @@ int arcb_launch_moe_route(const MoeArgs& a, cudaStream_t stream) {
   if (a.rows <= 0) return 0;
   if (a.experts > MOE_MAX_EXPERTS || a.top > MOE_MAX_TOP || a.top > a.experts || a.top < 1 || a.pitch % 8) return -1;
   if (a.max_slots < arcb_moe_max_slots(a.rows, a.experts, a.top, a.gran)) return -1;
-  const dim3 rows4((a.rows + 3) / 4);
-  cudaError_t e = !a.z ? arcb_launch(moe_router_kernel, dim3(a.rows), dim3(ROUTER_WARPS * 32), 0, stream, a)
-                  : a.experts <= 32  ? arcb_launch(moe_route_kernel<1>, rows4, dim3(128), 0, stream, a)
-                  : a.experts <= 64  ? arcb_launch(moe_route_kernel<2>, rows4, dim3(128), 0, stream, a)
-                  : a.experts <= 128 ? arcb_launch(moe_route_kernel<4>, rows4, dim3(128), 0, stream, a)
-                                     : arcb_launch(moe_route_kernel<8>, rows4, dim3(128), 0, stream, a);
+  auto go = [&](auto route, auto router) {
+    return a.z ? arcb_launch(route, dim3((a.rows + ROUTE_ROWS - 1) / ROUTE_ROWS), dim3(128), 0, stream, a)
+               : arcb_launch(router, dim3(a.rows), dim3(ROUTER_WARPS * 32), 0, stream, a);
+  };
+  cudaError_t e = a.experts <= 32    ? go(moe_route_kernel<1>, moe_router_kernel<1>)
+                  : a.experts <= 64  ? go(moe_route_kernel<2>, moe_router_kernel<2>)
+                  : a.experts <= 128 ? go(moe_route_kernel<4>, moe_router_kernel<4>)
+                                     : go(moe_route_kernel<8>, moe_router_kernel<8>);
   if (e != cudaSuccess) return (int)e;
   e = arcb_launch(moe_scatter_kernel, dim3(a.rows), dim3(SCATTER_THREADS), 0, stream, a);
   arcb_count_launch(2);
