@@ -14,6 +14,7 @@
 #include "attn_prefill_gqa.cuh"
 #include "engine.cuh"
 #include "gemm.cuh"
+#include "launch.cuh"
 #include "layerops.cuh"
 #include "mlstm.cuh"
 #include "moe.cuh"
@@ -120,6 +121,9 @@ struct LayeredSession {
   MoeArgs moe{};               // buffers
   void* moe_hid = nullptr;     // [max_slots][ffp]
   void* moe_out = nullptr;     // [max_slots][Wp]
+  // the shared expert of a decode step runs beside the routed ones
+  cudaStream_t side = nullptr;
+  cudaEvent_t fork = nullptr, join = nullptr;
 };
 
 namespace {
@@ -710,10 +714,20 @@ int lm_session_create(arcb_session* s) {
   }
   ls->expand = c;
   ls->expand_rows = lm_expand_rows(m, B, T);
+  if (m.has_moe) {
+    CK(cudaStreamCreateWithFlags(&ls->side, cudaStreamNonBlocking));
+    CK(cudaEventCreateWithFlags(&ls->fork, cudaEventDisableTiming));
+    CK(cudaEventCreateWithFlags(&ls->join, cudaEventDisableTiming));
+  }
   return ARCB_OK;
 }
 
-void lm_session_destroy(LayeredSession* ls) { delete ls; }
+void lm_session_destroy(LayeredSession* ls) {
+  if (ls->fork) cudaEventDestroy(ls->fork);
+  if (ls->join) cudaEventDestroy(ls->join);
+  if (ls->side) cudaStreamDestroy(ls->side);
+  delete ls;
+}
 int* lm_n_finished(arcb_session* s) { return s->ls->st.n_finished; }
 bool lm_armed(const arcb_session* s) { return s->ls->armed; }
 
@@ -856,6 +870,20 @@ int lm_mlp(arcb_session* s, int l, const Rows& R, cudaStream_t stream) {
     CKL(lm_gemm(m, ls->xn, L.w_up, eu, m.wp, stream), "gate/up gemm");
     return lm_residual(s, ls->hid, L.w_down, L.ffp, R.n, step, stream);
   }
+  // the shared expert: of a decode step, whose launches leave most of the GPU idle, on a stream of its own
+  if (L.sffp) {
+    const bool beside = step && ls->side && !arcb_pdl_enabled();
+    if (beside) {
+      CK(cudaEventRecord(ls->fork, stream));
+      CK(cudaStreamWaitEvent(ls->side, ls->fork, 0));
+    }
+    cudaStream_t st = beside ? ls->side : stream;
+    eu.N = 2 * L.sffp; eu.glu.limit = d.shared_limit;
+    CKL(lm_gemm(m, ls->xn, L.w_sgu, eu, m.wp, st), "shared gate/up gemm");
+    const int r = lm_residual(s, ls->hid, L.w_sdown, L.sffp, R.n, step, st);
+    if (r) return r;
+    if (beside) CK(cudaEventRecord(ls->join, ls->side));
+  }
   MoeArgs mo = ls->moe;
   mo.count += (size_t)l * MOE_MAX_EXPERTS;
   if (arcb_moe_router_inside(R.n, d.experts, m.wp, m.fmt)) {
@@ -878,10 +906,8 @@ int lm_mlp(arcb_session* s, int l, const Rows& R, cudaStream_t stream) {
   ed.mode = EPI_ACT; ed.M = slots; ed.N = m.wp; ed.out16 = ls->moe_out; ed.act_f16 = m.fmt; ed.err = s->eng->d_err;
   ed.grp.tile_group = mo.tile_expert; ed.grp.n_tiles = mo.n_tiles; ed.grp.group_rows = m.wp; ed.grp.w_rows = (long long)d.experts * m.wp;
   CKL(lm_gemm(m, ls->moe_hid, L.w_edown, ed, L.ffp, stream, variant), "expert down gemm");
-  if (!L.sffp) return ARCB_OK;
-  eu.N = 2 * L.sffp; eu.glu.limit = d.shared_limit;
-  CKL(lm_gemm(m, ls->xn, L.w_sgu, eu, m.wp, stream), "shared gate/up gemm");
-  return lm_residual(s, ls->hid, L.w_sdown, L.sffp, R.n, step, stream);
+  if (L.sffp && step && ls->side && !arcb_pdl_enabled()) CK(cudaStreamWaitEvent(stream, ls->join, 0));
+  return ARCB_OK;
 }
 
 int lm_mixer(arcb_session* s, int l, const Rows& R, cudaStream_t stream) {

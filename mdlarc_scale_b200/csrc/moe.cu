@@ -85,49 +85,61 @@ moe_route_kernel(MoeArgs a) {
   }
 }
 
-// One CTA of eight warps per row, which also multiplies the row with the router (16-bit formats).
-constexpr int ROUTER_WARPS = 8;
+// One CTA of eight warps per ROUTER_ROWS rows, which also multiplies the rows with the router (16-bit formats).
+constexpr int ROUTER_WARPS = 8, ROUTER_ROWS = 2;
 template <int PER_LANE>
 __global__ void __launch_bounds__(ROUTER_WARPS * 32)
 moe_router_kernel(MoeArgs a) {
   pdl_launch_dependents();
   pdl_wait();
-  __shared__ float s_z[MOE_MAX_EXPERTS];
-  const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const uint4* x = reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(a.xn) + (size_t)row * a.pitch);
+  __shared__ float s_z[ROUTER_ROWS][MOE_MAX_EXPERTS];
+  const int row0 = blockIdx.x * ROUTER_ROWS, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n = a.pitch / 8;                             // 8 columns a load
-  for (int e0 = warp * 4; e0 < a.experts; e0 += ROUTER_WARPS * 4) {
-    float d[4] = {0.f, 0.f, 0.f, 0.f};
-    const uint4* w = reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(a.w_router) + (size_t)e0 * a.pitch);
-#pragma unroll 4
-    for (int i = lane; i < n; i += 32) {                 // rows behind the last expert are zero
-      const uint4 xv = x[i];
-      const uint32_t xr[4] = {xv.x, xv.y, xv.z, xv.w};
+  const uint4* x[ROUTER_ROWS];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const uint4 wv = __ldg(w + (size_t)e * n + i);
-        const uint32_t wr[4] = {wv.x, wv.y, wv.z, wv.w};
+  for (int r = 0; r < ROUTER_ROWS; ++r)
+    x[r] = reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(a.xn) + (size_t)min(row0 + r, a.rows - 1) * a.pitch);
+  for (int e0 = warp * 4; e0 < a.experts; e0 += ROUTER_WARPS * 4) {
+    float d[ROUTER_ROWS][4] = {};
+    const uint4* w = reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(a.w_router) + (size_t)e0 * a.pitch);
+#pragma unroll 2
+    for (int i = lane; i < n; i += 32) {                 // rows behind the last expert are zero
+      uint4 wv[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) wv[e] = __ldg(w + (size_t)e * n + i);
+#pragma unroll
+      for (int r = 0; r < ROUTER_ROWS; ++r) {
+        const uint4 xv = x[r][i];
+        const uint32_t xr[4] = {xv.x, xv.y, xv.z, xv.w};
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-          const float2 p = unpack2_act(xr[j], a.fmt), q = unpack2_act(wr[j], a.fmt);
-          d[e] = fmaf(p.x, q.x, d[e]);
-          d[e] = fmaf(p.y, q.y, d[e]);
+          const float2 p = unpack2_act(xr[j], a.fmt);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const uint32_t wr[4] = {wv[e].x, wv[e].y, wv[e].z, wv[e].w};
+            const float2 q = unpack2_act(wr[j], a.fmt);
+            d[r][e] = fmaf(p.x, q.x, d[r][e]);
+            d[r][e] = fmaf(p.y, q.y, d[r][e]);
+          }
         }
       }
     }
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      d[e] = warp_sum(d[e]);
-      if (lane == 0 && e0 + e < a.experts) s_z[e0 + e] = d[e];
-    }
+    for (int r = 0; r < ROUTER_ROWS; ++r)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        d[r][e] = warp_sum(d[r][e]);
+        if (lane == 0 && e0 + e < a.experts) s_z[r][e0 + e] = d[r][e];
+      }
   }
   __syncthreads();
-  if (warp) return;
+  const int row = row0 + warp;
+  if (warp >= ROUTER_ROWS || row >= a.rows) return;
   float s[PER_LANE];
 #pragma unroll
   for (int i = 0; i < PER_LANE; ++i) {
     const int e = lane + 32 * i;
-    s[i] = e < a.experts ? score(s_z[e]) : -1.f;
+    s[i] = e < a.experts ? score(s_z[warp][e]) : -1.f;
   }
   float w;
   const int e = choose<PER_LANE>(a, lane, s, w);
@@ -218,7 +230,7 @@ int arcb_launch_moe_route(const MoeArgs& a, cudaStream_t stream) {
   if (a.max_slots < arcb_moe_max_slots(a.rows, a.experts, a.top, a.gran)) return -1;
   auto go = [&](auto route, auto router) {
     return a.z ? arcb_launch(route, dim3((a.rows + ROUTE_ROWS - 1) / ROUTE_ROWS), dim3(128), 0, stream, a)
-               : arcb_launch(router, dim3(a.rows), dim3(ROUTER_WARPS * 32), 0, stream, a);
+               : arcb_launch(router, dim3((a.rows + ROUTER_ROWS - 1) / ROUTER_ROWS), dim3(ROUTER_WARPS * 32), 0, stream, a);
   };
   cudaError_t e = a.experts <= 32    ? go(moe_route_kernel<1>, moe_router_kernel<1>)
                   : a.experts <= 64  ? go(moe_route_kernel<2>, moe_router_kernel<2>)
