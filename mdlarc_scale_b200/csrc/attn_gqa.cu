@@ -6,7 +6,8 @@ namespace {
 
 constexpr float LOG2E = 1.4426950408889634f;
 
-// One warp per (item, head): merges the splits in order, adds the sink, applies the gate.
+// One warp per (item, head): merges the splits in order, adds the sink, applies the gate.  Lane s keeps the factor of
+// splits s and s + 32.
 __global__ void __launch_bounds__(128)
 attn_gqa_combine_kernel(AttnGqaArgs a) {
   pdl_launch_dependents();
@@ -17,19 +18,41 @@ attn_gqa_combine_kernel(AttnGqaArgs a) {
   const int item = (int)(ih / a.n_heads), h = (int)(ih % a.n_heads);
   const int rec = a.vdimp + 4;
   const float* r0 = a.scratch + (size_t)ih * a.n_splits * rec;
+  float m_s[2], l_s[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int s = lane + 32 * i;
+    const float2 ml = s < a.n_splits ? *reinterpret_cast<const float2*>(r0 + (size_t)s * rec + a.vdimp) : make_float2(-INFINITY, 0.f);
+    m_s[i] = ml.x;
+    l_s[i] = ml.y;
+  }
   const float sk = a.sink ? a.sink[h] * LOG2E : -INFINITY;
-  float m = sk;
-  for (int s = 0; s < a.n_splits; ++s) m = fmaxf(m, r0[(size_t)s * rec + a.vdimp]);
+  float m = fmaxf(m_s[0], m_s[1]);
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+  m = fmaxf(m, sk);
   const float ms = (m == -INFINITY) ? 0.f : m;
-  float l = exp2f(sk - ms);
-  for (int s = 0; s < a.n_splits; ++s) l += r0[(size_t)s * rec + a.vdimp + 1] * exp2f(r0[(size_t)s * rec + a.vdimp] - ms);
+  const float f0 = exp2f(m_s[0] - ms), f1 = exp2f(m_s[1] - ms);
+  const float l = warp_sum(l_s[0] * f0 + l_s[1] * f1) + exp2f(sk - ms);
   const float inv = l > 0.f ? 1.f / l : 0.f;
-  for (int c = lane; c < a.vdimp; c += 32) {
-    float o = 0.f;
-    for (int s = 0; s < a.n_splits; ++s) o += r0[(size_t)s * rec + c] * exp2f(r0[(size_t)s * rec + a.vdimp] - ms);
-    o *= inv;
-    if (a.gate) o *= ld_act(a.gate, (size_t)item * a.gate_pitch + (size_t)h * a.vdimp + c, a.fmt);
-    st_act(a.out, (size_t)ih * a.vdimp + c, o, a.fmt);
+  for (int c = lane * 4; c < ((a.vdimp + 127) & ~127); c += 128) {       // every lane takes every step: the shuffles need them
+    const bool in = c < a.vdimp;
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int s = 0; s < a.n_splits; ++s) {
+      const float f = __shfl_sync(0xffffffffu, s < 32 ? f0 : f1, s & 31);
+      if (in) {
+        const float4 v = *reinterpret_cast<const float4*>(r0 + (size_t)s * rec + c);
+        o.x += v.x * f; o.y += v.y * f; o.z += v.z * f; o.w += v.w * f;
+      }
+    }
+    if (!in) continue;
+    o.x *= inv; o.y *= inv; o.z *= inv; o.w *= inv;
+    if (a.gate) {
+      const float4 g = ld_act4(a.gate, (size_t)item * a.gate_pitch + (size_t)h * a.vdimp + c, a.fmt);
+      o.x *= g.x; o.y *= g.y; o.z *= g.z; o.w *= g.w;
+    }
+    st_act4(a.out, (size_t)ih * a.vdimp + c, o, a.fmt);
   }
 }
 
