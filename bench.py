@@ -1026,8 +1026,8 @@ def main():
     ap.add_argument("--profile-decode-small", type=int, default=0, metavar="SEQS",
                     help="only run prefill + 15 decode steps of SEQS tiny prompts on a 64-position cache (ncu target)")
     ap.add_argument("--layered", choices=sorted(LAYERED_SIZES), default=None,
-                    help="prefill and decode throughput of a layered model (Vodavik) of this width beside a TinyTransformer "
-                         "of equal width and depth, instead of the headline workload")
+                    help="prefill and decode throughput of layered models of this width beside a TinyTransformer of equal "
+                         "width and depth, instead of the headline workload")
     ap.add_argument("--layered-layers", type=int, default=8)
     ap.add_argument("--layered-prompts", type=int, default=16, help="prompts of one prefill call")
     ap.add_argument("--layered-tokens", type=int, default=2048, help="tokens per prompt and decode context")
